@@ -4,6 +4,7 @@ from .viresun_config import ViresunConfig
 from .bivatar_config import BivatarConfig
 from .lazolix_config import LazolixConfig
 from .gezozen_config import GezozenConfig
+from .boketar_config import BoketarConfig
 
 __all__ = ["ConfigError", "LlamaConfig", "RopeScaling", "read_config_json", "EngineConfig", "ViresunConfig",
-           "BivatarConfig", "LazolixConfig", "GezozenConfig"]
+           "BivatarConfig", "LazolixConfig", "GezozenConfig", "BoketarConfig"]

@@ -55,7 +55,7 @@ __device__ __forceinline__ int awb_next_tile(int tile, int tiles_kept, int tile_
 // one warp per (row, head) of the stacked projection [q heads | k heads | v heads]; `bias` (or null) has one
 // number per column of the projection and is added as the sums are read; after the norm the first rot_dims
 // coordinates of every query and key head are turned by the row's cosine/sine pairs (coordinate i with
-// i + rot_dims/2); values are multiplied by value_scale on their way into the page
+// i + rot_dims/2, or 2i with 2i + 1 where `adjacent`); values are multiplied by value_scale on their way into the page
 template <typename TI, typename TA>
 __global__ void __launch_bounds__(QKN_THREADS)
 qk_norm_store_kernel(const TI* __restrict__ in, long long ld_in, TA* __restrict__ q_out, TA* __restrict__ cache,
@@ -63,7 +63,7 @@ qk_norm_store_kernel(const TI* __restrict__ in, long long ld_in, TA* __restrict_
                      const int* __restrict__ block_table, int max_blocks, int T, int nh, int nkv, int D, int VD, int P,
                      size_t page_stride, float eps, int normalise, float temp_coef, int temp_every,
                      const float* __restrict__ qw, const float* __restrict__ kw, const float* __restrict__ bias,
-                     const float* __restrict__ cos_sin, int rot_dims, float value_scale) {
+                     const float* __restrict__ cos_sin, int rot_dims, int adjacent, float value_scale) {
     __shared__ float turn_s[QKN_THREADS / 32][MAX_HEAD];
     const int lane = threadIdx.x & 31;
     const long long unit = (long long)blockIdx.x * (QKN_THREADS / 32) + (threadIdx.x >> 5);
@@ -112,7 +112,11 @@ qk_norm_store_kernel(const TI* __restrict__ in, long long ld_in, TA* __restrict_
 #pragma unroll
             for (int i = 0; i < MAX_HEAD / 32; ++i) {
                 const int d = lane + 32 * i;
-                if (d < rot_dims) {
+                if (d < rot_dims && adjacent) {
+                    // neighbouring lanes hold a pair (d and lane have the same parity)
+                    const float2 cs = *reinterpret_cast<const float2*>(cos_sin + ((size_t)t * half + d / 2) * 2);
+                    v[i] = (d & 1) == 0 ? v[i] * cs.x - mine[d + 1] * cs.y : v[i] * cs.x + mine[d - 1] * cs.y;
+                } else if (d < rot_dims) {
                     const int j = d < half ? d : d - half;
                     const float2 cs = *reinterpret_cast<const float2*>(cos_sin + ((size_t)t * half + j) * 2);
                     v[i] = d < half ? v[i] * cs.x - mine[d + half] * cs.y : v[i] * cs.x + mine[d - half] * cs.y;
@@ -140,8 +144,8 @@ AP_EXPORT int ap_qk_norm_store(const void* in, int in_dtype, long long ld_in, vo
                                const int* positions, const int* token_seq, const int* block_table, int max_blocks,
                                int T, int nh, int nkv, int D, int VD, int P, long long page_stride, float eps,
                                int normalise, float temp_coef, int temp_every, const float* qw, const float* kw,
-                               const float* bias, const float* cos_sin, int rot_dims, float value_scale,
-                               cudaStream_t stream) {
+                               const float* bias, const float* cos_sin, int rot_dims, int pairing,
+                               float value_scale, cudaStream_t stream) {
     AP_REQUIRE(T >= 0 && nh > 0 && nkv > 0 && D > 0 && VD > 0 && D <= MAX_HEAD && VD <= MAX_HEAD,
                "qk_norm_store: bad sizes T=%d heads=%d/%d sizes %d/%d (at most %d)", T, nh, nkv, D, VD, MAX_HEAD);
     AP_REQUIRE(cache == nullptr || (token_seq && block_table && max_blocks > 0 && P > 0),
@@ -149,6 +153,7 @@ AP_EXPORT int ap_qk_norm_store(const void* in, int in_dtype, long long ld_in, vo
     AP_REQUIRE(temp_every >= 0, "qk_norm_store: the temperature's period must not be negative");
     AP_REQUIRE(rot_dims == 0 || (cos_sin && rot_dims > 0 && rot_dims % 2 == 0 && rot_dims <= D),
                "qk_norm_store: %d rotated coordinates of %d need an even number and a table", rot_dims, D);
+    AP_REQUIRE(pairing == 0 || pairing == 1, "qk_norm_store: pairing %d is not known", pairing);
     if (T == 0) return AP_OK;
     const long long units = (long long)T * (nh + 2 * nkv);
     const dim3 grid((unsigned)((units + QKN_THREADS / 32 - 1) / (QKN_THREADS / 32)));
@@ -157,7 +162,7 @@ AP_EXPORT int ap_qk_norm_store(const void* in, int in_dtype, long long ld_in, vo
                         ap_launch_pdl(qk_norm_store_kernel<TI, TA>, grid, dim3(QKN_THREADS), 0, stream, (const TI*)in, \
                                       ld_in, (TA*)q_out, (TA*)cache, positions, token_seq, block_table, max_blocks, T, \
                                       nh, nkv, D, VD, P, (size_t)page_stride, eps, normalise, temp_coef, temp_every, \
-                                      qw, kw, bias, cos_sin, rot_dims, value_scale))
+                                      qw, kw, bias, cos_sin, rot_dims, pairing == 1 ? 1 : 0, value_scale))
     if (in_dtype == AP_F32 && act_dtype == AP_F32) LAUNCH(float, float);
     else if (in_dtype == AP_F32 && act_dtype == AP_BF16) LAUNCH(float, bf16);
     else if (in_dtype == AP_BF16 && act_dtype == AP_BF16) LAUNCH(bf16, bf16);

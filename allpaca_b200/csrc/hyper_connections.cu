@@ -1,0 +1,231 @@
+// Hyper-connections: the residual is not one vector per row but `streams` of them, x_1 .. x_n.  A sublayer reads one
+// weighted sum of the streams and its result goes back to all of them, while they also mix among themselves:
+//
+//   y     = scale * sum_s rmsnorm(delta[s] + bias[s]) * slice_w[s]      or plainly  sum_s (delta[s] + bias[s])
+//   x_t  <- sum_s mix[s][t] x_s + out_w[t] y                            (all streams at once from the old ones)
+//   u     = sum_s in_w[s] x_s                                           (the NEXT reader's weights)
+//   out   = rmsnorm(u) * w
+//
+// One kernel does what lies between two sublayers: it finishes the sublayer before (its pending sums, possibly the
+// results of two mixers side by side, each normed on its own), brings the streams up to date and norms what the next
+// sublayer reads.  Without `mix` the old streams do not enter (the first reader of a step: all streams start as
+// copies of the embedding row, which is then the pending result).  Without a pending result the streams stay as they
+// are.  With chosen rows only those are produced and the streams are left alone: the model's last norm.
+//
+// All 32-bit up to the store of `out`.  One CTA per row; sums over a row are formed in a fixed order that depends on
+// the width alone, so a row has the same bits in any batch.
+#include "common.cuh"
+
+#define HC_MAX_STREAMS 32
+#define HC_MAX_SLICES 4
+
+struct StreamNormArgs {
+    float* x;                        // [T][streams][H]
+    const int* rows;                 // chosen rows, or null
+    const float* delta; int S; size_t slice_stride;          // pending sums [S][T][H], or null
+    const float* slice_bias;         // [S][H] or null
+    const float* slice_w;            // [S][H] or null: every slice over its own root mean square, times this
+    float slice_eps, slice_scale;
+    const float* out_w;              // [streams]
+    const float* mix;                // [streams from][streams to] or null
+    const float* in_w;               // [streams]
+    const float* w; float eps;       // the norm's weight [H]
+    int update;                      // the streams are brought up to date
+    int streams, H;
+};
+
+template <int VEC> __device__ __forceinline__ void hc_load(const float* p, float (&v)[VEC]) {
+    if constexpr (VEC == 4) {
+        const float4 t = *reinterpret_cast<const float4*>(p);
+        v[0] = t.x; v[1] = t.y; v[2] = t.z; v[3] = t.w;
+    } else {
+        v[0] = p[0];
+    }
+}
+template <int VEC> __device__ __forceinline__ void hc_store(float* p, const float (&v)[VEC]) {
+    if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    else p[0] = v[0];
+}
+template <int VEC> __device__ __forceinline__ void hc_store(bf16* p, const float (&v)[VEC]) {
+    if constexpr (VEC == 4) {
+        const __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+        uint2 t;
+        t.x = *reinterpret_cast<const unsigned*>(&a);
+        t.y = *reinterpret_cast<const unsigned*>(&b);
+        *reinterpret_cast<uint2*>(p) = t;
+    } else {
+        p[0] = __float2bfloat16_rn(v[0]);
+    }
+}
+
+// NS: the number of streams the kernel is built for (0: any number up to HC_MAX_STREAMS)
+template <int NS, int VEC, typename TO>
+__global__ void stream_norm_kernel(const StreamNormArgs A, TO* __restrict__ out) {
+    constexpr int N = NS ? NS : HC_MAX_STREAMS;
+    extern __shared__ __align__(16) float u_s[];             // [H]
+    __shared__ float scratch[32];
+    __shared__ float mix_s[N * N], out_s[N], in_s[N];
+    const int n = NS ? NS : A.streams;
+    ap_pdl_trigger();
+    // the weights do not depend on earlier kernels
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+        out_s[i] = A.out_w ? A.out_w[i] : 0.f;
+        in_s[i] = A.in_w[i];
+    }
+    if (A.mix) for (int i = threadIdx.x; i < n * n; i += blockDim.x) mix_s[i] = A.mix[i];
+    ap_pdl_wait();
+    const int H = A.H;
+    const size_t t = A.rows ? (size_t)A.rows[blockIdx.x] : (size_t)blockIdx.x;
+    float* xr = A.x + t * n * H;
+    const float* dr = A.delta ? A.delta + t * H : nullptr;
+    const bool reads_old = A.delta == nullptr || A.mix != nullptr;
+    float factor[HC_MAX_SLICES];
+#pragma unroll
+    for (int s = 0; s < HC_MAX_SLICES; ++s) factor[s] = 1.0f;
+    if (dr && A.slice_w) {
+#pragma unroll
+        for (int s = 0; s < HC_MAX_SLICES; ++s) {
+            if (s >= A.S) break;
+            float ss = 0.f;
+            for (int c = threadIdx.x * VEC; c < H; c += blockDim.x * VEC) {
+                float d[VEC], b[VEC];
+                hc_load<VEC>(dr + s * A.slice_stride + c, d);
+                if (A.slice_bias) {
+                    hc_load<VEC>(A.slice_bias + (size_t)s * H + c, b);
+#pragma unroll
+                    for (int i = 0; i < VEC; ++i) d[i] += b[i];
+                }
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) ss = fmaf(d[i], d[i], ss);
+            }
+            ss = ap_block_sum(ss, scratch);
+            factor[s] = A.slice_scale / sqrtf(ss / (float)H + A.slice_eps);
+        }
+    }
+    __syncthreads();                                         // the weights are in shared memory
+    float ss = 0.f;
+    for (int c = threadIdx.x * VEC; c < H; c += blockDim.x * VEC) {
+        float old[N][VEC], u[VEC];
+        if (reads_old) {
+#pragma unroll(NS ? N : 1)
+            for (int s = 0; s < N; ++s)
+                if (s < n) hc_load<VEC>(xr + (size_t)s * H + c, old[s]);
+        }
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) u[i] = 0.f;
+        if (dr) {
+            float y[VEC];
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) y[i] = 0.f;
+#pragma unroll
+            for (int s = 0; s < HC_MAX_SLICES; ++s) {
+                if (s >= A.S) break;
+                float d[VEC], b[VEC];
+                hc_load<VEC>(dr + s * A.slice_stride + c, d);
+                if (A.slice_bias) {
+                    hc_load<VEC>(A.slice_bias + (size_t)s * H + c, b);
+#pragma unroll
+                    for (int i = 0; i < VEC; ++i) d[i] += b[i];
+                }
+                if (A.slice_w) {
+                    hc_load<VEC>(A.slice_w + (size_t)s * H + c, b);
+#pragma unroll
+                    for (int i = 0; i < VEC; ++i) d[i] = d[i] * factor[s] * b[i];
+                }
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) y[i] += d[i];
+            }
+#pragma unroll(NS ? N : 1)
+            for (int o = 0; o < N; ++o) {
+                if (o >= n) break;
+                float v[VEC];
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) v[i] = out_s[o] * y[i];
+                if (A.mix) {
+#pragma unroll(NS ? N : 1)
+                    for (int s = 0; s < N; ++s) {
+                        if (s >= n) break;
+                        const float m = mix_s[s * n + o];
+#pragma unroll
+                        for (int i = 0; i < VEC; ++i) v[i] = fmaf(m, old[s][i], v[i]);
+                    }
+                }
+                if (A.update) hc_store<VEC>(xr + (size_t)o * H + c, v);
+                const float wi = in_s[o];
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) u[i] = fmaf(wi, v[i], u[i]);
+            }
+        } else {
+#pragma unroll(NS ? N : 1)
+            for (int s = 0; s < N; ++s) {
+                if (s >= n) break;
+                const float wi = in_s[s];
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) u[i] = fmaf(wi, old[s][i], u[i]);
+            }
+        }
+        hc_store<VEC>(u_s + c, u);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) ss = fmaf(u[i], u[i], ss);
+    }
+    ss = ap_block_sum(ss, scratch);
+    const float inv = 1.0f / sqrtf(ss / (float)H + A.eps);
+    // a thread reads back the columns it wrote itself
+    for (int c = threadIdx.x * VEC; c < H; c += blockDim.x * VEC) {
+        float u[VEC], ww[VEC];
+        hc_load<VEC>(u_s + c, u);
+        hc_load<VEC>(A.w + c, ww);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) u[i] = u[i] * inv * ww[i];
+        hc_store<VEC>(out + (size_t)blockIdx.x * H + c, u);
+    }
+}
+
+AP_EXPORT int ap_stream_norm(float* x, const int* rows, int R, const float* delta, int S, long long slice_stride,
+                             const float* slice_bias, const float* slice_w, float slice_eps, float slice_scale,
+                             const float* out_w, const float* mix, const float* in_w, const float* w, float eps,
+                             int update, void* out, int out_dtype, int streams, int H, cudaStream_t stream) {
+    AP_REQUIRE(R >= 0 && H > 0 && x && in_w && w && out, "stream_norm: bad arguments R=%d H=%d", R, H);
+    AP_REQUIRE(streams >= 1 && streams <= HC_MAX_STREAMS, "stream_norm: %d streams are not in 1..%d", streams, HC_MAX_STREAMS);
+    AP_REQUIRE(delta == nullptr || (S >= 1 && S <= HC_MAX_SLICES && out_w), "stream_norm: %d slices of pending sums are not "
+               "in 1..%d, or the streams' weights on them are missing", S, HC_MAX_SLICES);
+    AP_REQUIRE(!(update && rows), "stream_norm: chosen rows leave the streams alone");
+    if (R == 0) return AP_OK;
+    const bool vec = H % 4 == 0 && slice_stride % 4 == 0 &&
+                     ((((uintptr_t)x) | ((uintptr_t)delta) | ((uintptr_t)slice_bias) | ((uintptr_t)slice_w) | ((uintptr_t)w)) & 15) == 0 &&
+                     (((uintptr_t)out) & (out_dtype == AP_F32 ? 15 : 7)) == 0;
+    int threads = ((vec ? H / 4 : H) + 31) / 32 * 32;
+    if (threads > 512) threads = 512;
+    const size_t smem = (size_t)H * sizeof(float);
+    AP_REQUIRE(smem <= 200 * 1024, "stream_norm: a row of %d does not fit shared memory", H);
+    StreamNormArgs A;
+    A.x = x; A.rows = rows; A.delta = delta; A.S = delta ? S : 0; A.slice_stride = (size_t)slice_stride;
+    A.slice_bias = slice_bias; A.slice_w = slice_w; A.slice_eps = slice_eps; A.slice_scale = slice_scale;
+    A.out_w = out_w; A.mix = mix; A.in_w = in_w; A.w = w; A.eps = eps; A.update = (update && delta) ? 1 : 0;
+    A.streams = streams; A.H = H;
+#define LAUNCH(N, V, TO)                                                                                            \
+    do {                                                                                                            \
+        auto kern = stream_norm_kernel<N, V, TO>;                                                                   \
+        if (smem > 40 * 1024) {                                                                                     \
+            cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
+            AP_REQUIRE(e == cudaSuccess, "stream_norm: cannot reserve %zu bytes of shared memory", smem);           \
+        }                                                                                                           \
+        AP_CHECK_PDL_LAUNCH("stream_norm", ap_launch_pdl(kern, dim3((unsigned)R), dim3(threads), smem, stream, A, (TO*)out)); \
+    } while (0)
+#define LAUNCH_T(N, V) do { if (out_dtype == AP_F32) LAUNCH(N, V, float); else LAUNCH(N, V, bf16); } while (0)
+#define LAUNCH_V(N) do { if (vec) LAUNCH_T(N, 4); else LAUNCH_T(N, 1); } while (0)
+    AP_REQUIRE(out_dtype == AP_F32 || out_dtype == AP_BF16, "stream_norm: unknown dtype %d", out_dtype);
+    switch (streams) {
+        case 1: LAUNCH_V(1); break;
+        case 2: LAUNCH_V(2); break;
+        case 3: LAUNCH_V(3); break;
+        case 4: LAUNCH_V(4); break;
+        case 6: LAUNCH_V(6); break;
+        case 8: LAUNCH_V(8); break;
+        default: LAUNCH_T(0, 1);
+    }
+#undef LAUNCH_V
+#undef LAUNCH_T
+#undef LAUNCH
+    return AP_OK;
+}

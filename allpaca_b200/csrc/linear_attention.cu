@@ -6,15 +6,18 @@
 // with the variants as parameters of one kernel:
 //   decay a_t   one fixed number per head (DECAY_HEAD_CONST: retention);
 //               one number per head and token, exp(-exp(A_log[h]) * softplus(raw + dt_bias[h])) (DECAY_HEAD_TOKEN);
-//               one number per key channel and token, sigmoid(z)^(1/tau) = exp(-softplus(-z) / tau) (DECAY_CHANNEL)
+//               one number per key channel and token, sigmoid(z)^(1/tau) = exp(-softplus(-z) / tau) (DECAY_CHANNEL),
+//               or exp(-exp(A_log[h]) * softplus(z + dt_bias[h, channel])) (DECAY_CHANNEL_TOKEN)
 //   write u_t   the value v_t; or, with the delta rule, beta_t (v_t - S^T k_t) with S already decayed and
 //               beta_t = sigmoid(raw), so that the read-out sees the corrected state
 //   q, k        as projected (QK_PLAIN); the first rot_dims coordinates of every head turned by the step's
 //               cosine/sine table, coordinate i with i + rot_dims/2 (QK_ROTATE); or made unit vectors,
-//               x / sqrt(sum x^2 + unit_eps) (QK_UNIT).  Several value heads may share a query/key head.
+//               x / sqrt(sum x^2 + unit_eps) (QK_UNIT); or, like the values, under SiLU (QKV_SILU).  Several value
+//               heads may share a query/key head.
 //
-// and the kernel that finishes a head's read-out: RMS over the head (a weight per coordinate or none), times
-// silu(gate), times a constant, rounded to the activation type for the output projection.
+// and the kernel that finishes a head's read-out: RMS over the head, or over all heads together (a weight per
+// coordinate or none), times silu(gate) or sigmoid(gate), times a constant, rounded to the activation type for the
+// output projection.
 //
 // Everything is 32-bit: inputs are 32-bit sums of the projections, decays, exponentials, the state, the
 // read-out and the norm.  A sequence's rows are found through seq_start, its state row through
@@ -27,9 +30,11 @@
 #define DECAY_HEAD_CONST 0
 #define DECAY_HEAD_TOKEN 1
 #define DECAY_CHANNEL 2
+#define DECAY_CHANNEL_TOKEN 3
 #define QK_PLAIN 0
 #define QK_ROTATE 1
 #define QK_UNIT 2
+#define QKV_SILU 3
 
 __device__ __forceinline__ float la_softplus(float v) { return v > 20.0f ? v : log1pf(expf(v)); }
 __device__ __forceinline__ float la_silu(float v) { return v / (1.0f + expf(-v)); }
@@ -45,11 +50,11 @@ __device__ __forceinline__ void la_copy16(float* dst, const float* src) {
 struct LaScanArgs {
     float* q; long long ld_q;                  // head g of row t: q[t * ld_q + g * D + d]; made ready in place
     float* k; long long ld_k;
-    const float* v; long long ld_v;            // head h of row t: v[t * ld_v + h * V + c]
-    float* decay_channel; long long ld_dc;     // DECAY_CHANNEL: z[t * ld_dc + h * D + d], becomes the decay in place
+    float* v; long long ld_v;                  // head h of row t: v[t * ld_v + h * V + c]; QKV_SILU: in place
+    float* decay_channel; long long ld_dc;     // DECAY_CHANNEL*: z[t * ld_dc + h * D + d], becomes the decay in place
     float* decay_head; long long ld_dh;        // DECAY_HEAD_TOKEN: raw[t * ld_dh + h], becomes the decay in place
-    const float* decay_const;                  // DECAY_HEAD_CONST: the decay [heads]; DECAY_HEAD_TOKEN: A_log [heads]
-    const float* dt_bias;                      // DECAY_HEAD_TOKEN: [heads] or null
+    const float* decay_const;                  // DECAY_HEAD_CONST: the decay [heads]; DECAY_*_TOKEN: A_log [heads]
+    const float* dt_bias;                      // DECAY_HEAD_TOKEN: [heads], DECAY_CHANNEL_TOKEN: [heads * D]; or null
     float* beta; long long ld_beta;            // raw[t * ld_beta + h], becomes sigmoid in place; null: no delta rule
     const float* cos_sin; int rot_dims;        // QK_ROTATE: [T, rot_dims / 2, 2]
     float* state; long long state_stride;      // [slots][heads][D][V]
@@ -61,17 +66,18 @@ struct LaScanArgs {
 
 // What has to happen to a step's rows before the recurrence reads them, once per row and in place (the
 // recurrence's CTAs share a head's queries and keys, so none of this belongs into them): one warp per
-// (row, unit) with the units of a row being its query heads, its key heads (rotation or unit vectors), its heads'
-// channel decays (exp(-softplus(-z) / tau)) and one unit for the numbers per head (decay and sigmoid(beta)).
+// (row, unit) with the units of a row being its query heads, its key heads (rotation, unit vectors or SiLU), its
+// value heads (SiLU), its heads' channel decays and one unit for the numbers per head (decay and sigmoid(beta)).
 __global__ void __launch_bounds__(128) la_prepare_kernel(const LaScanArgs A) {
     ap_pdl_trigger();
     ap_pdl_wait();
     const int lane = threadIdx.x & 31;
     const int G = A.qk_heads, H = A.heads, D = A.D;
     const int qk_units = A.qk_mode == QK_PLAIN ? 0 : 2 * G;
-    const int ch_units = A.decay_mode == DECAY_CHANNEL ? H : 0;
+    const int v_units = A.qk_mode == QKV_SILU ? H : 0;
+    const int ch_units = A.decay_mode >= DECAY_CHANNEL ? H : 0;
     const int sc_units = (A.decay_mode == DECAY_HEAD_TOKEN || A.beta != nullptr) ? 1 : 0;
-    const int units = qk_units + ch_units + sc_units;
+    const int units = qk_units + v_units + ch_units + sc_units;
     const long long unit = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
     if (unit >= (long long)A.T * units) return;
     const int t = (int)(unit / units);
@@ -86,6 +92,8 @@ __global__ void __launch_bounds__(128) la_prepare_kernel(const LaScanArgs A) {
                 p[j] = a * cs.x - b * cs.y;
                 p[j + half] = b * cs.x + a * cs.y;
             }
+        } else if (A.qk_mode == QKV_SILU) {
+            for (int d = lane; d < D; d += 32) p[d] = la_silu(p[d]);
         } else {
             float ss = 0.f;
             for (int d = lane; d < D; d += 32) ss = fmaf(p[d], p[d], ss);
@@ -96,9 +104,21 @@ __global__ void __launch_bounds__(128) la_prepare_kernel(const LaScanArgs A) {
         return;
     }
     u -= qk_units;
+    if (u < v_units) {
+        float* p = A.v + (size_t)t * A.ld_v + (size_t)u * A.V;
+        for (int d = lane; d < A.V; d += 32) p[d] = la_silu(p[d]);
+        return;
+    }
+    u -= v_units;
     if (u < ch_units) {
         float* z = A.decay_channel + (size_t)t * A.ld_dc + (size_t)u * D;
-        for (int d = lane; d < D; d += 32) z[d] = expf(-la_softplus(-z[d]) * A.inv_tau);
+        if (A.decay_mode == DECAY_CHANNEL) {
+            for (int d = lane; d < D; d += 32) z[d] = expf(-la_softplus(-z[d]) * A.inv_tau);
+        } else {
+            const float rate = expf(A.decay_const[u]);
+            const float* b = A.dt_bias ? A.dt_bias + (size_t)u * D : nullptr;
+            for (int d = lane; d < D; d += 32) z[d] = expf(-rate * la_softplus(z[d] + (b ? b[d] : 0.f)));
+        }
         return;
     }
     for (int h = lane; h < H; h += 32) {
@@ -136,7 +156,7 @@ __global__ void __launch_bounds__(128) la_scan_kernel(const LaScanArgs A) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
     const int vcol = col0 + vl;
     const bool live = vl < ncols;
-    const bool channel = A.decay_mode == DECAY_CHANNEL, delta = A.beta != nullptr;
+    const bool channel = A.decay_mode >= DECAY_CHANNEL, delta = A.beta != nullptr;
     const bool token_decay = A.decay_mode == DECAY_HEAD_TOKEN;
     const int XS = (cols + 3) / 4 * 4, DS = PER * NP;        // a row of keys in shared memory is padded with zeros
     // one buffer: v [CHUNK][XS], k [CHUNK][DS], q [CHUNK][DS], channel decays [CHUNK][DS] (if any), decay [CHUNK], beta [CHUNK]
@@ -275,7 +295,7 @@ __global__ void __launch_bounds__(128) la_scan_kernel(const LaScanArgs A) {
     }
 }
 
-AP_EXPORT int ap_linear_scan(float* q, long long ld_q, float* k, long long ld_k, const float* v,
+AP_EXPORT int ap_linear_scan(float* q, long long ld_q, float* k, long long ld_k, float* v,
                              long long ld_v, float* decay_channel, long long ld_dc, float* decay_head,
                              long long ld_dh, const float* decay_const, const float* dt_bias, float* beta,
                              long long ld_beta, const float* cos_sin, int rot_dims, float* state,
@@ -290,9 +310,10 @@ AP_EXPORT int ap_linear_scan(float* q, long long ld_q, float* k, long long ld_k,
                "linear_scan: an operand is missing or the state is too small");
     AP_REQUIRE(decay_mode == DECAY_HEAD_CONST ? decay_const != nullptr
                : decay_mode == DECAY_HEAD_TOKEN ? (decay_head != nullptr && decay_const != nullptr)
-               : (decay_mode == DECAY_CHANNEL && decay_channel != nullptr && tau > 0.f),
+               : decay_mode == DECAY_CHANNEL ? (decay_channel != nullptr && tau > 0.f)
+               : (decay_mode == DECAY_CHANNEL_TOKEN && decay_channel != nullptr && decay_const != nullptr),
                "linear_scan: decay mode %d lacks its numbers", decay_mode);
-    AP_REQUIRE(qk_mode == QK_PLAIN || qk_mode == QK_UNIT ||
+    AP_REQUIRE(qk_mode == QK_PLAIN || qk_mode == QK_UNIT || qk_mode == QKV_SILU ||
                (qk_mode == QK_ROTATE && cos_sin && rot_dims > 0 && rot_dims % 2 == 0 && rot_dims <= D),
                "linear_scan: query/key mode %d with %d rotated coordinates of %d", qk_mode, rot_dims, D);
     if (T == 0 || nseq == 0) return AP_OK;
@@ -315,7 +336,7 @@ AP_EXPORT int ap_linear_scan(float* q, long long ld_q, float* k, long long ld_k,
     auto aligned = [](const void* p, long long ld) { return p == nullptr || ((((uintptr_t)p) & 15) == 0 && ld % 4 == 0); };
     const int vec = (D % 4 == 0 && V % 4 == 0 && cols % 4 == 0 && aligned(q, ld_q) && aligned(k, ld_k) &&
                      aligned(v, ld_v) && aligned(decay_channel, ld_dc)) ? 1 : 0;
-    const bool channel = decay_mode == DECAY_CHANNEL;
+    const bool channel = decay_mode >= DECAY_CHANNEL;
     LaScanArgs A;
     A.q = q; A.ld_q = ld_q; A.k = k; A.ld_k = ld_k; A.v = v; A.ld_v = ld_v;
     A.decay_channel = decay_channel; A.ld_dc = ld_dc; A.decay_head = decay_head; A.ld_dh = ld_dh;
@@ -324,8 +345,8 @@ AP_EXPORT int ap_linear_scan(float* q, long long ld_q, float* k, long long ld_k,
     A.seq_start = seq_start; A.positions = positions; A.state_slots = state_slots; A.y = y; A.ld_y = ld_y;
     A.T = T; A.heads = heads; A.qk_heads = qk_heads; A.D = D; A.V = V; A.NP = NP; A.cols = cols;
     A.decay_mode = decay_mode; A.qk_mode = qk_mode; A.vec = vec;
-    A.inv_tau = channel ? 1.0f / tau : 0.f; A.unit_eps = unit_eps; A.out_scale = out_scale;
-    const int units = (qk_mode == QK_PLAIN ? 0 : 2 * qk_heads) + (channel ? heads : 0) +
+    A.inv_tau = decay_mode == DECAY_CHANNEL ? 1.0f / tau : 0.f; A.unit_eps = unit_eps; A.out_scale = out_scale;
+    const int units = (qk_mode == QK_PLAIN ? 0 : 2 * qk_heads) + (qk_mode == QKV_SILU ? heads : 0) + (channel ? heads : 0) +
                       ((decay_mode == DECAY_HEAD_TOKEN || beta != nullptr) ? 1 : 0);
     if (units > 0) {
         const long long blocks = ((long long)T * units + 3) / 4;
@@ -352,41 +373,52 @@ AP_EXPORT int ap_linear_scan(float* q, long long ld_q, float* k, long long ld_k,
 }
 
 // ---- a head's read-out: RMS norm, gate, constant ------------------------------------------
-// y: [T, ld_y] 32-bit, head h at column h * V; gate: [T, ld_g] 32-bit raw, same layout; one warp per (row, head).
-template <typename TO>
-__global__ void __launch_bounds__(128)
+// y: [T, ld_y] 32-bit, head h at column h * V; gate: [T, ld_g] 32-bit raw, same layout; `threads` (a warp, or a CTA
+// where the heads are long: a norm over all heads together is one head of their whole width) per (row, head).
+#define GATE_SILU 0
+#define GATE_SIGMOID 1
+#define HNG_THREADS 128
+
+template <typename TO, bool WHOLE_CTA>
+__global__ void __launch_bounds__(HNG_THREADS)
 head_norm_gate_kernel(const float* __restrict__ y, long long ld_y, const float* __restrict__ gate, long long ld_g,
-                      const float* __restrict__ w, float eps, float out_scale, TO* __restrict__ out, int T, int heads,
-                      int V) {
+                      const float* __restrict__ w, float eps, float out_scale, int act, TO* __restrict__ out, int T,
+                      int heads, int V) {
+    __shared__ float scratch[32];
     ap_pdl_trigger();
     ap_pdl_wait();
-    const long long unit = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
-    if (unit >= (long long)T * heads) return;
-    const int lane = threadIdx.x & 31;
+    const long long unit = WHOLE_CTA ? (long long)blockIdx.x : (long long)blockIdx.x * (HNG_THREADS / 32) + (threadIdx.x >> 5);
+    if (unit >= (long long)T * heads) return;                // (a whole CTA always has its unit)
+    const int first = WHOLE_CTA ? threadIdx.x : (threadIdx.x & 31), stride = WHOLE_CTA ? HNG_THREADS : 32;
     const int t = (int)(unit / heads), h = (int)(unit % heads);
     const float* yr = y + (size_t)t * ld_y + (size_t)h * V;
     const float* gr = gate + (size_t)t * ld_g + (size_t)h * V;
     float ss = 0.f;
-    for (int i = lane; i < V; i += 32) ss = fmaf(yr[i], yr[i], ss);
-    ss = ap_warp_sum(ss);
+    for (int i = first; i < V; i += stride) ss = fmaf(yr[i], yr[i], ss);
+    ss = WHOLE_CTA ? ap_block_sum(ss, scratch) : ap_warp_sum(ss);
     const float inv = out_scale / sqrtf(ss / (float)V + eps);
     TO* o = out + ((size_t)t * heads + h) * V;
-    for (int i = lane; i < V; i += 32)
-        o[i] = ap_from_float<TO>(yr[i] * inv * (w ? w[i] : 1.0f) * la_silu(gr[i]));
+    for (int i = first; i < V; i += stride) {
+        const float s = 1.0f / (1.0f + expf(-gr[i]));
+        o[i] = ap_from_float<TO>(yr[i] * inv * (w ? w[i] : 1.0f) * (act == GATE_SILU ? gr[i] * s : s));
+    }
 }
 
 AP_EXPORT int ap_head_norm_gate(const float* y, long long ld_y, const float* gate, long long ld_g, const float* w,
-                                float eps, float out_scale, void* out, int out_dtype, int T, int heads, int V,
+                                float eps, float out_scale, int act, void* out, int out_dtype, int T, int heads, int V,
                                 cudaStream_t stream) {
     AP_REQUIRE(T >= 0 && heads > 0 && V > 0 && ld_y >= (long long)heads * V && ld_g >= (long long)heads * V,
                "head_norm_gate: bad sizes heads=%d value=%d", heads, V);
+    AP_REQUIRE(act == GATE_SILU || act == GATE_SIGMOID, "head_norm_gate: gate %d is not known", act);
     if (T == 0) return AP_OK;
-    const dim3 grid((unsigned)(((long long)T * heads + 3) / 4));
-#define LAUNCH(TO)                                                                                                  \
-    AP_CHECK_PDL_LAUNCH("head_norm_gate", ap_launch_pdl(head_norm_gate_kernel<TO>, grid, dim3(128), 0, stream, y,   \
-                                                        ld_y, gate, ld_g, w, eps, out_scale, (TO*)out, T, heads, V))
-    if (out_dtype == AP_F32) LAUNCH(float);
-    else if (out_dtype == AP_BF16) LAUNCH(bf16);
+    const bool whole = V > 256;
+    const long long units = (long long)T * heads, per = whole ? 1 : HNG_THREADS / 32;
+    const dim3 grid((unsigned)((units + per - 1) / per));
+#define LAUNCH(TO, WHOLE)                                                                                           \
+    AP_CHECK_PDL_LAUNCH("head_norm_gate", ap_launch_pdl(head_norm_gate_kernel<TO, WHOLE>, grid, dim3(HNG_THREADS), 0, stream, \
+                                                        y, ld_y, gate, ld_g, w, eps, out_scale, act, (TO*)out, T, heads, V))
+    if (out_dtype == AP_F32) { if (whole) LAUNCH(float, true); else LAUNCH(float, false); }
+    else if (out_dtype == AP_BF16) { if (whole) LAUNCH(bf16, true); else LAUNCH(bf16, false); }
     else AP_REQUIRE(false, "head_norm_gate: unknown dtype %d", out_dtype);
 #undef LAUNCH
     return AP_OK;

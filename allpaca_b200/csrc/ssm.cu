@@ -1,8 +1,8 @@
 // A selective state-space mixer in its recurrent form (state-space duality, one scalar decay
 // per head), with the state a request carries from step to step:
 //
-//   causal_conv_silu   u_t[c] = silu(b[c] + sum_j w[c][j] * in_{t-(taps-1)+j}[c])     (in_t = 0 for t < 0)
-//   conv_state_update  the last taps-1 inputs of every sequence, for its next step
+//   causal_conv        u_t[c] = act(b[c] + sum_j w[c][j] * in_{t-(taps-1)+j}[c])      (in_t = 0 for t < 0; act:
+//                      SiLU or none), and the last taps-1 inputs of every sequence kept for its next step
 //   ssm_scan           dt = softplus(raw + dt_bias[h]);  S_t = exp(-exp(A_log[h]) dt) S_{t-1} + dt B_t x_t^T;
 //                      y_t = S_t^T C_t + D[h] x_t                                        (S: [N, vdim] per head)
 //   gated_group_rmsnorm  out = rmsnorm_per_group(y * silu(z)) * w
@@ -17,84 +17,147 @@
 __device__ __forceinline__ float ssm_silu(float v) { return v / (1.0f + expf(-v)); }
 __device__ __forceinline__ float ssm_softplus(float v) { return v > 20.0f ? v : log1pf(expf(v)); }
 
-// ---- causal convolution per channel, with SiLU -----------------------------------------
-// in: [T, ld_in] 32-bit, the convolved channels start at column `col0`; out: [T, C] 32-bit.
-// state: [slots][taps-1][C] 32-bit, the inputs at positions first-(taps-1) .. first-1.
-__global__ void causal_conv_silu_kernel(const float* __restrict__ in, long long ld_in, int col0,
-                                        const float* __restrict__ w, const float* __restrict__ bias,
-                                        const float* __restrict__ state, long long state_stride,
-                                        const int* __restrict__ token_seq, const int* __restrict__ seq_start,
-                                        const int* __restrict__ positions, const int* __restrict__ state_slots,
-                                        float* __restrict__ out, int T, int C, int taps) {
-    ap_pdl_trigger();
-    ap_pdl_wait();
-    const size_t n = (size_t)T * C;
-    for (size_t e = blockIdx.x * (size_t)blockDim.x + threadIdx.x; e < n; e += (size_t)gridDim.x * blockDim.x) {
-        const int t = (int)(e / C), c = (int)(e - (size_t)t * C);
-        const int s = token_seq[t];
-        const int first_row = seq_start[s];
-        const int pos = positions[t];
-        const int local = t - first_row;                       // row of the sequence's portion
-        const float* st = state + (size_t)state_slots[s] * state_stride;
-        float a = bias ? bias[c] : 0.f;
-        for (int j = 0; j < taps; ++j) {
-            const int back = taps - 1 - j;                     // how many tokens before this one
-            float v = 0.f;
-            if (pos - back >= 0) {
-                if (local - back >= 0) v = in[(size_t)(t - back) * ld_in + col0 + c];
-                else v = st[(size_t)(taps - 1 + (local - back)) * C + c];
-            }
-            a = fmaf(w[(size_t)c * taps + j], v, a);
-        }
-        out[e] = ssm_silu(a);
+// ---- causal convolution per channel ------------------------------------------------------
+// in: [T, ld_in] 32-bit, the convolved channels start at column `col0`; in_bias (or null) is added to an input
+// before it is filtered (a bias of the product that made it); out: [T, C] 32-bit, activated or as filtered.
+// state: [slots][taps-1][C] 32-bit, the (biased) inputs at positions first-(taps-1) .. first-1.
+//
+// One thread takes VEC channels of a run of consecutive rows of ONE sequence's portion and slides a window of
+// taps-1 inputs over them, so that every input is read about once.  Runs start at the portion's first row and
+// have at least taps-1 rows, so only the thread of a portion's first run ever reads the request's state; the same
+// thread brings the state up to date afterwards, which no other thread can miss.
+// TAPS 0: any number of taps, inputs read again for every tap.
+#define CONV_ROWS 8
+#define CONV_THREADS 128
+#define CONV_ACT_NONE 0
+#define CONV_ACT_SILU 1
+
+template <int VEC> __device__ __forceinline__ void conv_load(const float* p, const float* bias, float (&v)[VEC]) {
+    if constexpr (VEC == 4) {
+        const float4 t = *reinterpret_cast<const float4*>(p);
+        v[0] = t.x; v[1] = t.y; v[2] = t.z; v[3] = t.w;
+    } else {
+        v[0] = p[0];
     }
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] += bias[i];
 }
 
-__global__ void conv_state_update_kernel(const float* __restrict__ in, long long ld_in, int col0,
-                                         float* __restrict__ state, long long state_stride,
-                                         const int* __restrict__ seq_start, const int* __restrict__ positions,
-                                         const int* __restrict__ state_slots, int C, int taps) {
+template <int TAPS, int VEC>
+__global__ void __launch_bounds__(CONV_THREADS)
+causal_conv_kernel(const float* __restrict__ in, long long ld_in, int col0, const float* __restrict__ in_bias,
+                   const float* __restrict__ w, const float* __restrict__ bias, int act, float* state,
+                   long long state_stride, const int* __restrict__ seq_start, const int* __restrict__ positions,
+                   const int* __restrict__ state_slots, float* __restrict__ out, int nseq, int C, int taps_rt, int run) {
     ap_pdl_trigger();
     ap_pdl_wait();
-    const int s = blockIdx.x;
-    const int a = seq_start[s], n = seq_start[s + 1] - a;
-    if (n <= 0) return;
+    const int taps = TAPS ? TAPS : taps_rt, keep = taps - 1;
+    const int c = (blockIdx.y * CONV_THREADS + threadIdx.x) * VEC;
+    int b = blockIdx.x, seq = -1, a = 0, n = 0;
+    for (int s = 0; s < nseq; ++s) {
+        a = seq_start[s];
+        n = seq_start[s + 1] - a;
+        const int runs = (n + run - 1) / run;
+        if (b < runs) { seq = s; break; }
+        b -= runs;
+    }
+    if (seq < 0 || c >= C) return;
+    const int r0 = b * run, rows = min(run, n - r0);          // rows r0 .. of the sequence's portion
     const int first_pos = positions[a];
-    float* st = state + (size_t)state_slots[s] * state_stride;
-    const int keep = taps - 1;
-    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < C; c += gridDim.y * blockDim.x) {
-        // slot k holds the input `keep - k` tokens before the next step's first one; ascending k
-        // reads old slots only at higher indices than it has written
+    float* st = keep > 0 ? state + (size_t)state_slots[seq] * state_stride + c : nullptr;
+    const float* src = in + col0 + c;
+    float ib[VEC], ob[VEC];
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) { ib[i] = in_bias ? in_bias[c + i] : 0.f; ob[i] = bias ? bias[c + i] : 0.f; }
+    // the input `r` rows into the portion (r < 0: from the request's state, or nothing before the start)
+    auto input = [&](int r, float (&v)[VEC]) {
+        if (r >= 0) {
+            conv_load<VEC>(src + (size_t)(a + r) * ld_in, ib, v);
+        } else {
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) v[i] = first_pos + r >= 0 ? st[(size_t)(keep + r) * C + i] : 0.f;
+        }
+    };
+    if constexpr (TAPS > 0) {
+        float ww[TAPS][VEC], win[TAPS][VEC];                  // win[j]: the input taps-1-j tokens before the row
+#pragma unroll
+        for (int i = 0; i < VEC; ++i)
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) ww[j][i] = w[(size_t)(c + i) * TAPS + j];
+#pragma unroll
+        for (int j = 0; j + 1 < TAPS; ++j) input(r0 - (TAPS - 1) + j, win[j]);
+#pragma unroll 4
+        for (int r = r0; r < r0 + rows; ++r) {
+            conv_load<VEC>(src + (size_t)(a + r) * ld_in, ib, win[TAPS - 1]);
+            float v[VEC];
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) {
+                v[i] = ob[i];
+#pragma unroll
+                for (int j = 0; j < TAPS; ++j) v[i] = fmaf(ww[j][i], win[j][i], v[i]);
+                if (act == CONV_ACT_SILU) v[i] = ssm_silu(v[i]);
+#pragma unroll
+                for (int j = 0; j + 1 < TAPS; ++j) win[j][i] = win[j + 1][i];
+            }
+            float* o = out + (size_t)(a + r) * C + c;
+            if constexpr (VEC == 4) *reinterpret_cast<float4*>(o) = make_float4(v[0], v[1], v[2], v[3]);
+            else o[0] = v[0];
+        }
+    } else {
+        for (int r = r0; r < r0 + rows; ++r) {
+            float v[VEC], x[VEC];
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) v[i] = ob[i];
+            for (int j = 0; j < taps; ++j) {
+                input(r - keep + j, x);
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) v[i] = fmaf(w[(size_t)(c + i) * taps + j], x[i], v[i]);
+            }
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) out[(size_t)(a + r) * C + c + i] = act == CONV_ACT_SILU ? ssm_silu(v[i]) : v[i];
+        }
+    }
+    if (b == 0) {
+        // slot k holds the input `keep - k` tokens before the next step's first one; ascending k reads old slots
+        // only at higher indices than it has written
         for (int k = 0; k < keep; ++k) {
-            const int local = n - keep + k;                    // row of this portion, < 0: from before it
-            float v;
-            if (local >= 0) v = in[(size_t)(a + local) * ld_in + col0 + c];
-            else if (first_pos + local >= 0) v = st[(size_t)(keep + local) * C + c];
-            else v = 0.f;
-            st[(size_t)k * C + c] = v;
+            float v[VEC];
+            input(n - keep + k, v);
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) st[(size_t)k * C + i] = v[i];
         }
     }
 }
 
-AP_EXPORT int ap_causal_conv_silu(const float* in, long long ld_in, int col0, const float* w, const float* bias,
-                                  float* state, long long state_stride, const int* token_seq, const int* seq_start,
-                                  const int* positions, const int* state_slots, float* out, int T, int nseq, int C,
-                                  int taps, cudaStream_t stream) {
-    AP_REQUIRE(T >= 0 && nseq >= 0 && C > 0 && taps >= 1 && ld_in >= col0 + C, "causal_conv_silu: bad sizes");
-    AP_REQUIRE(taps == 1 || state != nullptr, "causal_conv_silu: a convolution over several tokens needs its state");
-    if (T == 0) return AP_OK;
-    long long blocks = ((long long)T * C + 255) / 256;
-    if (blocks > 148 * 16) blocks = 148 * 16;
-    AP_CHECK_PDL_LAUNCH("causal_conv_silu",
-                        ap_launch_pdl(causal_conv_silu_kernel, dim3((unsigned)blocks), dim3(256), 0, stream, in, ld_in,
-                                      col0, w, bias, (const float*)state, state_stride, token_seq, seq_start, positions,
-                                      state_slots, out, T, C, taps));
-    if (taps > 1 && nseq > 0) {
-        const dim3 grid((unsigned)nseq, (unsigned)((C + 255) / 256));
-        AP_CHECK_PDL_LAUNCH("conv_state_update",
-                            ap_launch_pdl(conv_state_update_kernel, grid, dim3(256), 0, stream, in, ld_in, col0, state,
-                                          state_stride, seq_start, positions, state_slots, C, taps));
+AP_EXPORT int ap_causal_conv(const float* in, long long ld_in, int col0, const float* in_bias, const float* w,
+                             const float* bias, int act, float* state, long long state_stride, const int* seq_start,
+                             const int* positions, const int* state_slots, float* out, int T, int nseq, int C, int taps,
+                             cudaStream_t stream) {
+    AP_REQUIRE(T >= 0 && nseq >= 0 && C > 0 && taps >= 1 && ld_in >= col0 + C, "causal_conv: bad sizes");
+    AP_REQUIRE(act == CONV_ACT_NONE || act == CONV_ACT_SILU, "causal_conv: activation %d is not known", act);
+    AP_REQUIRE(taps == 1 || state != nullptr, "causal_conv: a convolution over several tokens needs its state");
+    if (T == 0 || nseq == 0) return AP_OK;
+    const int run = taps - 1 > CONV_ROWS ? taps - 1 : CONV_ROWS;
+    const bool vec = C % 4 == 0 && col0 % 4 == 0 && ld_in % 4 == 0 && ((((uintptr_t)in) | ((uintptr_t)out)) & 15) == 0 &&
+                     taps <= 6;
+    const int per = CONV_THREADS * (vec ? 4 : 1);
+    const dim3 grid((unsigned)(T / run + nseq), (unsigned)((C + per - 1) / per));
+#define LAUNCH(N, V)                                                                                                \
+    AP_CHECK_PDL_LAUNCH("causal_conv", ap_launch_pdl(causal_conv_kernel<N, V>, grid, dim3(CONV_THREADS), 0, stream, in, \
+                                                     ld_in, col0, in_bias, w, bias, act, state, state_stride, seq_start, \
+                                                     positions, state_slots, out, nseq, C, taps, run))
+#define LAUNCH_V(N) do { if (vec) LAUNCH(N, 4); else LAUNCH(N, 1); } while (0)
+    switch (taps) {
+        case 1: LAUNCH_V(1); break;
+        case 2: LAUNCH_V(2); break;
+        case 3: LAUNCH_V(3); break;
+        case 4: LAUNCH_V(4); break;
+        case 5: LAUNCH_V(5); break;
+        case 6: LAUNCH_V(6); break;
+        default: LAUNCH(0, 1);
     }
+#undef LAUNCH_V
+#undef LAUNCH
     return AP_OK;
 }
 

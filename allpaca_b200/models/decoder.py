@@ -18,7 +18,8 @@ from typing import Dict, List, Mapping, Optional, Tuple
 import torch
 
 from .. import ops
-from ..parts import (Block, BuildEnv, CacheNeed, Deferred, LayerCache, ModelSpec, Part, WeightSpec, build)
+from ..parts import (Block, BuildEnv, CacheNeed, Deferred, LayerCache, ModelSpec, Part, Slices, StreamUpdate,
+                     WeightSpec, build)
 from ..parts.linear import Linear
 
 
@@ -38,6 +39,7 @@ class DecoderModel:
         self.final_norm = build("norm", spec.final_norm, env)
         self.embedding_norm = build("norm", spec.embedding_norm, env) if spec.embedding_norm is not None else None
         self._sinusoid_inv_freq: Optional[torch.Tensor] = None
+        self._stream_ones: Optional[torch.Tensor] = None      # a weight of 1 per residual stream
         self.embedding: Optional[torch.Tensor] = None
         self.head = Linear(env, spec.vocab_size, spec.hidden_size)
         self.head_bias: Optional[torch.Tensor] = None
@@ -89,6 +91,8 @@ class DecoderModel:
         for block in self.blocks:
             block.finalize()
         s = self.spec
+        if s.streams is not None:
+            self._stream_ones = torch.ones(s.streams, dtype=torch.float32, device=self.env.device)
         self.embedding = tensors[s.embedding_name].contiguous()
         if s.tie_word_embeddings or s.head_name not in tensors:
             # tied by flag, or by absence as the reference does (model.rs:8006-8009)
@@ -168,17 +172,22 @@ class DecoderModel:
         for g, (pages, page_dim) in enumerate(self._group_pages):
             ops.clear_page_tails(pages, page_dim, step.positions, step.token_seq, step.block_tables[g],
                                  step.context_lens)
-        x = ws.get("model.residual", (T, s.hidden_size), torch.float32)
+        if s.streams is None:
+            x = embedded = ws.get("model.residual", (T, s.hidden_size), torch.float32)
+        else:
+            # the streams start as copies of the embedding row: it is the first reader's pending result
+            x = ws.get("model.residual", (T, s.streams, s.hidden_size), torch.float32)
+            embedded = ws.get("model.embedded", (T, s.hidden_size), torch.float32)
         scale = s.embedding_scale if s.embedding_scale is not None else 1.0
         if s.embedding_sinusoid_base is not None or self.embedding_norm is not None:
             # position vector and norm of the embedding row in the kernel that gathers it
             norm = self.embedding_norm
             ops.embed_sinusoid_norm(step.token_ids, step.positions, self.embedding, self._sinusoid_frequencies(),
                                     norm.weight if norm is not None else None, norm.eps if norm is not None else 0.0,
-                                    x, scale)
+                                    embedded, scale)
         else:
-            ops.embed_gather(step.token_ids, self.embedding, x, scale)
-        delta = None
+            ops.embed_gather(step.token_ids, self.embedding, embedded, scale)
+        delta = None if s.streams is None else StreamUpdate(Slices(embedded.unsqueeze(0)), self._stream_ones)
         for r, run in enumerate(s.order):
             delta = self.blocks[run.layer].forward(x, delta, step, self.caches[r])
         R = step.num_logit_rows
@@ -188,7 +197,10 @@ class DecoderModel:
         h = ws.get("model.final_normed", (R, s.hidden_size), self.env.dtype)
         if isinstance(delta, Deferred):
             delta = None                 # the last block has added into the residual itself
-        self.final_norm.forward(x, h, delta=delta, rows=step.logit_rows)
+        if s.streams is None:
+            self.final_norm.forward(x, h, delta=delta, rows=step.logit_rows)
+        else:
+            self.final_norm.forward_streams(x, self._stream_ones, h, pending=delta, rows=step.logit_rows)
         out = self.head.forward(h, "model.logits", "float32")
         if self.head_bias is not None or s.logit_scale is not None or s.logit_softcap:
             ops.logit_transform(out, self.head_bias, s.logit_scale if s.logit_scale is not None else 1.0,

@@ -43,9 +43,9 @@ _CORE_SIGNATURES = {
     "ap_embed_sinusoid_norm": [_P, _P, _P, _I, _P, _P, _I, _F, _F, _P, _I, _I, _I, _P],
     # int ap_qk_norm_store(in, in_dtype, ld_in, q_out, cache, act_dtype, positions, token_seq, block_table,
     #                      max_blocks, T, nh, nkv, D, VD, P, page_stride, eps, normalise, temp_coef, temp_every,
-    #                      q_weight, k_weight, bias, cos_sin, rot_dims, value_scale, stream)
+    #                      q_weight, k_weight, bias, cos_sin, rot_dims, pairing, value_scale, stream)
     "ap_qk_norm_store": [_P, _I, _L, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _L, _F, _I, _F, _I, _P, _P, _P,
-                         _P, _I, _F, _P],
+                         _P, _I, _I, _F, _P],
     # int ap_attention_window_bias(q, out, cache, dtype, block_table, max_blocks, seq_start, positions, nseq, T,
     #                              nh, nkv, D, VD, P, page_stride, scale, softcap, window, r1, r2, single_rows,
     #                              other_rows, record, value_offset, bias_kind, keep_first, gate, gate_ld, sink,
@@ -70,9 +70,9 @@ _CORE_SIGNATURES = {
     #                       gate_ld, window, sink, stream)
     "ap_latent_prefill": [_P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _P, _L, _I, _P, _P],
     "ap_latent_prefill_takes": [_I, _I],
-    # int ap_causal_conv_silu(in, ld_in, col0, w, bias, state, state_stride, token_seq, seq_start, positions,
-    #                         state_slots, out, T, nseq, C, taps, stream)
-    "ap_causal_conv_silu": [_P, _L, _I, _P, _P, _P, _L, _P, _P, _P, _P, _P, _I, _I, _I, _I, _P],
+    # int ap_causal_conv(in, ld_in, col0, in_bias, w, bias, act, state, state_stride, seq_start, positions,
+    #                    state_slots, out, T, nseq, C, taps, stream)
+    "ap_causal_conv": [_P, _L, _I, _P, _P, _P, _I, _P, _L, _P, _P, _P, _P, _I, _I, _I, _I, _P],
     # int ap_ssm_scan(xbc, ld_xbc, dt_raw, ld_dt, dt_bias, a_log, d_skip, state, state_stride, seq_start, positions,
     #                 state_slots, y, T, nseq, heads, groups, N, vdim, stream)
     "ap_ssm_scan": [_P, _L, _P, _L, _P, _P, _P, _P, _L, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
@@ -106,8 +106,11 @@ _CORE_SIGNATURES = {
     #                    T, nseq, heads, qk_heads, D, V, decay_mode, qk_mode, tau, unit_eps, out_scale, stream)
     "ap_linear_scan": [_P, _L, _P, _L, _P, _L, _P, _L, _P, _L, _P, _P, _P, _L, _P, _I, _P, _L, _P, _P, _P, _P, _L,
                        _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _P],
-    # int ap_head_norm_gate(y, ld_y, gate, ld_g, w, eps, out_scale, out, out_dtype, T, heads, V, stream)
-    "ap_head_norm_gate": [_P, _L, _P, _L, _P, _F, _F, _P, _I, _I, _I, _I, _P],
+    # int ap_head_norm_gate(y, ld_y, gate, ld_g, w, eps, out_scale, act, out, out_dtype, T, heads, V, stream)
+    "ap_head_norm_gate": [_P, _L, _P, _L, _P, _F, _F, _I, _P, _I, _I, _I, _I, _P],
+    # int ap_stream_norm(x, rows, R, delta, S, slice_stride, slice_bias, slice_w, slice_eps, slice_scale, out_w, mix,
+    #                    in_w, w, eps, update, out, out_dtype, streams, H, stream)
+    "ap_stream_norm": [_P, _P, _I, _P, _I, _L, _P, _P, _F, _F, _P, _P, _P, _P, _F, _I, _P, _I, _I, _I, _P],
     # int ap_gated_postnorm(x, rows, R, delta, S, slice_stride, gate, ld_gate, gate_bias, alpha, w, w_dtype, groups,
     #                       eps, update, out, out_dtype, H, stream)
     "ap_gated_postnorm": [_P, _P, _I, _P, _I, _L, _P, _L, _P, _F, _P, _I, _I, _F, _I, _P, _I, _I, _P],

@@ -61,7 +61,7 @@ def qk_norm_store(qkv: torch.Tensor, q_out: torch.Tensor, cache_layer: Optional[
                   normalise: bool = True, temp_coef: float = 0.0, temp_every: int = 0,
                   q_weight: Optional[torch.Tensor] = None, k_weight: Optional[torch.Tensor] = None,
                   bias: Optional[torch.Tensor] = None, cos_sin: Optional[torch.Tensor] = None,
-                  value_scale: float = 1.0) -> None:
+                  pairing: int = 0, value_scale: float = 1.0) -> None:
     """Prepare the operands of :func:`attention_window_bias` from the stacked projection
     ``qkv [T, nh*D + nkv*D + nkv*VD (+ more columns that are not read)]``: every query and key head
     rescaled to unit mean square (``normalise``) and multiplied by ``q_weight`` / ``k_weight``
@@ -70,7 +70,7 @@ def qk_norm_store(qkv: torch.Tensor, q_out: torch.Tensor, cache_layer: Optional[
     ``q_out [T, nh*D]``, keys and values into the pages ``cache_layer [pages, nkv, P, D + VD]``
     (None: not stored).  ``bias`` (32-bit, one number per column of Q, K and V) is added to the sums as they are
     read; ``cos_sin [T, r/2, 2]`` turns the first ``r`` coordinates of every normed query and key head, coordinate
-    ``i`` with ``i + r/2``; values are multiplied by ``value_scale`` on their way into the page."""
+    ``i`` with ``i + r/2`` (``pairing`` 0) or ``2i`` with ``2i + 1`` (1); values are multiplied by ``value_scale`` on their way into the page."""
     if qkv.dim() != 2 or not qkv.is_cuda or qkv.stride(1) != 1:
         raise KernelError("qk_norm_store: qkv must be a CUDA matrix with contiguous rows")
     _check(q_out, "q_out", dims=2)
@@ -108,7 +108,7 @@ def qk_norm_store(qkv: torch.Tensor, q_out: torch.Tensor, cache_layer: Optional[
          value_dim, P, page_stride, float(eps), 1 if normalise else 0, float(temp_coef), int(temp_every),
          q_weight.data_ptr() if q_weight is not None else 0, k_weight.data_ptr() if k_weight is not None else 0,
          bias.data_ptr() if bias is not None else 0, cos_sin.data_ptr() if cos_sin is not None else 0, rot_dims,
-         float(value_scale), stream_handle())
+         int(pairing), float(value_scale), stream_handle())
 
 
 def attention_window_bias(q: torch.Tensor, out: torch.Tensor, cache_layer: torch.Tensor, block_table: torch.Tensor,
@@ -258,32 +258,42 @@ def head_project(inp: torch.Tensor, weight: Optional[torch.Tensor], out: torch.T
          int(tail), int(tail_dims), csptr, stream_handle())
 
 
-def causal_conv_silu(inp: torch.Tensor, col0: int, weight: torch.Tensor, bias: Optional[torch.Tensor],
-                     state: Optional[torch.Tensor], token_seq: torch.Tensor, seq_start: torch.Tensor,
-                     positions: torch.Tensor, state_slots: torch.Tensor, out: torch.Tensor, num_seqs: int) -> None:
-    """``out[t, c] = silu(bias[c] + sum_j weight[c, j] * in[t - (taps-1) + j, col0 + c])`` per
-    sequence, inputs of negative positions being zero; ``state [slots, taps-1, C]`` (32-bit, may be a strided
-    view of the slots' rows) supplies the inputs from before the step and is brought up to date."""
+CONV_ACTIVATIONS = {None: 0, "silu": 1}
+
+
+def causal_conv(inp: torch.Tensor, col0: int, weight: torch.Tensor, bias: Optional[torch.Tensor],
+                state: Optional[torch.Tensor], seq_start: torch.Tensor, positions: torch.Tensor,
+                state_slots: torch.Tensor, out: torch.Tensor, num_seqs: int, activation: Optional[str] = "silu",
+                in_bias: Optional[torch.Tensor] = None) -> None:
+    """``out[t, c] = act(bias[c] + sum_j weight[c, j] * (in[t - (taps-1) + j, col0 + c] + in_bias[c]))`` per
+    sequence, inputs of negative positions being zero (without the bias); ``activation``: ``"silu"`` or None.
+    ``state [slots, taps-1, C]`` (32-bit, may be a strided view of the slots' rows) supplies the biased inputs from
+    before the step and is brought up to date."""
     _check(inp, "in", torch.float32, 2)
     _check(weight, "weight", torch.float32, 2)
     _check(out, "out", torch.float32, 2)
     T, C = out.shape
     taps = weight.shape[1]
     if weight.shape[0] != C or inp.shape[0] < T or inp.shape[1] < col0 + C:
-        raise KernelError("causal_conv_silu: shapes disagree")
-    if bias is not None:
-        _check(bias, "bias", torch.float32, 1)
+        raise KernelError("causal_conv: shapes disagree")
+    if activation not in CONV_ACTIVATIONS:
+        raise KernelError(f"causal_conv: activation {activation!r} is not known")
+    for b, n in ((bias, "bias"), (in_bias, "in_bias")):
+        if b is not None:
+            _check(b, n, torch.float32, 1)
+            if b.shape[0] != C:
+                raise KernelError(f"causal_conv: {n} must have one entry per channel")
     sptr, sstride = 0, 0
     if taps > 1:
         if state is None or state.dtype != torch.float32 or state.dim() != 3 \
                 or tuple(state.shape[1:]) != (taps - 1, C) or state.stride(2) != 1 or state.stride(1) != C:
-            raise KernelError("causal_conv_silu: the state must be 32-bit [slots, taps-1, C] with contiguous rows")
+            raise KernelError("causal_conv: the state must be 32-bit [slots, taps-1, C] with contiguous rows")
         sptr, sstride = state.data_ptr(), state.stride(0)
-    for t, n in ((token_seq, "token_seq"), (seq_start, "seq_start"), (positions, "positions"),
-                 (state_slots, "state_slots")):
+    for t, n in ((seq_start, "seq_start"), (positions, "positions"), (state_slots, "state_slots")):
         _check(t, n, torch.int32, 1)
-    call(core(), "ap_causal_conv_silu", inp.data_ptr(), inp.stride(0), int(col0), weight.data_ptr(),
-         bias.data_ptr() if bias is not None else 0, sptr, sstride, token_seq.data_ptr(), seq_start.data_ptr(),
+    call(core(), "ap_causal_conv", inp.data_ptr(), inp.stride(0), int(col0),
+         in_bias.data_ptr() if in_bias is not None else 0, weight.data_ptr(),
+         bias.data_ptr() if bias is not None else 0, CONV_ACTIVATIONS[activation], sptr, sstride, seq_start.data_ptr(),
          positions.data_ptr(), state_slots.data_ptr(), out.data_ptr(), T, int(num_seqs), C, taps, stream_handle())
 
 

@@ -8,8 +8,9 @@ import torch
 
 from . import AP_F32, KernelError, _check, _partials, call, core, dtype_code, stream_handle
 
-DECAY_MODES = {"head": 0, "head_token": 1, "channel": 2}
-QK_MODES = {None: 0, "plain": 0, "rotate": 1, "unit": 2}
+DECAY_MODES = {"head": 0, "head_token": 1, "channel": 2, "channel_token": 3}
+QK_MODES = {None: 0, "plain": 0, "rotate": 1, "unit": 2, "silu": 3}
+GATE_ACTIVATIONS = {"silu": 0, "sigmoid": 1}
 
 
 def _rows32(t: torch.Tensor, name: str, T: int, width: int):
@@ -36,13 +37,16 @@ def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, y: torch.Tens
     ``q``, ``k`` ``[T, qk_heads * key_dim]``, ``v`` ``[T, heads * value_dim]`` (views of columns of a wider
     32-bit matrix are taken); value head ``h`` reads query/key head ``h // (heads / qk_heads)``.
     ``decay``: ``"head"``: ``a = decay_const[h]``; ``"head_token"``: ``a = exp(-exp(decay_const[h]) *
-    softplus(decay_head[t, h] + dt_bias[h]))``; ``"channel"``: ``a[d] = sigmoid(decay_channel[t, h, d])^(1/tau)``.
+    softplus(decay_head[t, h] + dt_bias[h]))``; ``"channel"``: ``a[d] = sigmoid(decay_channel[t, h, d])^(1/tau)``;
+    ``"channel_token"``: ``a[d] = exp(-exp(decay_const[h]) * softplus(decay_channel[t, h, d] + dt_bias[h, d]))``.
     ``beta [T, heads]`` (raw): the delta rule, ``u = sigmoid(beta) (v - S^T k)`` on the decayed state; else
     ``u = v``.  ``qk``: ``"rotate"`` turns the first ``2 * cos_sin.shape[1]`` coordinates of every query and key
-    head by ``cos_sin [T, r/2, 2]``; ``"unit"`` divides each by ``sqrt(sum x^2 + unit_eps)``.
+    head by ``cos_sin [T, r/2, 2]``; ``"unit"`` divides each by ``sqrt(sum x^2 + unit_eps)``; ``"silu"`` puts queries,
+    keys AND values under SiLU.
     ``state [slots, heads, key_dim, value_dim]`` may be a strided view of the slots' rows; a sequence whose first
-    row has position 0 starts from zero.  ``q``, ``k``, ``decay_channel``, ``decay_head`` and ``beta`` are scratch:
-    a pass before the recurrence turns them into what it reads (rotated or unit vectors, decays, gates) in place."""
+    row has position 0 starts from zero.  ``q``, ``k``, ``v``, ``decay_channel``, ``decay_head`` and ``beta`` are
+    scratch: a pass before the recurrence turns them into what it reads (rotated, unit or activated vectors, decays,
+    gates) in place."""
     T = y.shape[0]
     if decay not in DECAY_MODES or qk not in QK_MODES:
         raise KernelError(f"linear_scan: decay {decay!r} or qk {qk!r} is not known")
@@ -51,16 +55,18 @@ def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, y: torch.Tens
     vp, ldv = _rows32(v, "v", T, heads * value_dim)
     yp, ldy = _rows32(y, "y", T, heads * value_dim)
     dcp = dcl = dhp = dhl = bp = bl = 0
-    if decay == "channel":
+    if decay in ("channel", "channel_token"):
         dcp, dcl = _rows32(decay_channel, "decay_channel", T, heads * key_dim)
     if decay == "head_token":
         dhp, dhl = _rows32(decay_head, "decay_head", T, heads)
-    if decay in ("head", "head_token"):
+    if decay != "channel":
         _check(decay_const, "decay_const", torch.float32, 1)
         if decay_const.shape[0] != heads:
             raise KernelError("linear_scan: one decay constant per head is needed")
     if dt_bias is not None:
         _check(dt_bias, "dt_bias", torch.float32, 1)
+        if dt_bias.shape[0] != (heads * key_dim if decay == "channel_token" else heads):
+            raise KernelError("linear_scan: dt_bias must have one entry per decay")
     if beta is not None:
         bp, bl = _rows32(beta, "beta", T, heads)
     rot = 0
@@ -84,10 +90,14 @@ def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, y: torch.Tens
 
 
 def head_norm_gate(y: torch.Tensor, gate: torch.Tensor, weight: Optional[torch.Tensor], eps: float,
-                   out: torch.Tensor, heads: int, value_dim: int, out_scale: float = 1.0) -> None:
-    """``out[t, h] = y[t, h] / sqrt(mean(y[t, h]^2) + eps) * weight * silu(gate[t, h]) * out_scale`` per head of
+                   out: torch.Tensor, heads: int, value_dim: int, out_scale: float = 1.0,
+                   activation: str = "silu") -> None:
+    """``out[t, h] = y[t, h] / sqrt(mean(y[t, h]^2) + eps) * weight * act(gate[t, h]) * out_scale`` per head of
     ``value_dim`` numbers; ``y`` and ``gate`` 32-bit ``[T, heads * value_dim]`` (may be runs of columns of a
-    wider matrix), ``weight`` 32-bit ``[value_dim]`` shared by the heads or None."""
+    wider matrix), ``weight`` 32-bit ``[value_dim]`` shared by the heads or None; ``activation`` ``"silu"`` or
+    ``"sigmoid"``.  A norm over several heads together is one head of their whole width."""
+    if activation not in GATE_ACTIVATIONS:
+        raise KernelError(f"head_norm_gate: gate activation {activation!r} is not known")
     T = out.shape[0]
     _check(out, "out", dims=2)
     yp, ldy = _rows32(y, "y", T, heads * value_dim)
@@ -99,7 +109,8 @@ def head_norm_gate(y: torch.Tensor, gate: torch.Tensor, weight: Optional[torch.T
         if weight.shape[0] != value_dim:
             raise KernelError("head_norm_gate: the weight must have one entry per coordinate of a head")
     call(core(), "ap_head_norm_gate", yp, ldy, gp, ldg, weight.data_ptr() if weight is not None else 0, float(eps),
-         float(out_scale), out.data_ptr(), dtype_code(out.dtype), T, int(heads), int(value_dim), stream_handle())
+         float(out_scale), GATE_ACTIVATIONS[activation], out.data_ptr(), dtype_code(out.dtype), T, int(heads),
+         int(value_dim), stream_handle())
 
 
 def gated_postnorm(x: torch.Tensor, weight: torch.Tensor, groups: int, eps: float, alpha: float = 1.0,

@@ -1,6 +1,7 @@
-"""Python faces of the kernels that act on the residual stream element by element: a norm without
-statistics (Dynamic Tanh), its mix with the previous token's row, the depth-weighted average over
-the layers' outputs, and bias with activation behind a product; see ``ops/__init__.py``."""
+"""Python faces of the kernels that act on the residual stream: a norm without statistics (Dynamic
+Tanh), its mix with the previous token's row, the depth-weighted average over the layers' outputs, the
+streams of hyper-connections with the norm that reads them, and bias with activation behind a product;
+see ``ops/__init__.py``."""
 from __future__ import annotations
 
 from typing import Optional
@@ -88,6 +89,50 @@ def stream_mix(x: torch.Tensor, delta: Optional[torch.Tensor], streams: torch.Te
             raise KernelError("stream_mix: one weight per stream is needed")
     call(core(), "ap_stream_mix", x.data_ptr(), dptr, S, dstride, streams.data_ptr(), streams.stride(0), int(k),
          weights.data_ptr() if weights is not None else 0, x.numel(), stream_handle())
+
+
+def stream_norm(x: torch.Tensor, in_w: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor,
+                delta: Optional[torch.Tensor] = None, out_w: Optional[torch.Tensor] = None,
+                mix: Optional[torch.Tensor] = None, slice_bias: Optional[torch.Tensor] = None,
+                slice_weight: Optional[torch.Tensor] = None, slice_eps: float = 0.0, slice_scale: float = 1.0,
+                rows: Optional[torch.Tensor] = None) -> None:
+    """What lies between two sublayers of a decoder whose residual is ``n`` streams, ``x [T, n, H]`` (32-bit):
+    finish the pending result ``y``, bring the streams up to date, ``x_t = sum_s mix[s, t] x_s + out_w[t] y``, and
+    norm the weighted sum the next sublayer reads, ``out = rmsnorm(sum_s in_w[s] x_s) * weight``.
+
+    ``delta [S, T, H]`` (32-bit, up to four slices): ``y = sum_s (delta[s] + slice_bias[s])`` or, with
+    ``slice_weight [S, H]``, ``slice_scale * sum_s rmsnorm(delta[s] + slice_bias[s]) * slice_weight[s]``, each slice
+    over its own root mean square (``slice_eps``).  ``mix [n, n]`` (from, to) None: the old streams do not enter (all
+    become ``out_w[t] y``).  ``delta`` None: nothing is pending and the streams stay.  With ``rows`` (int32 indices)
+    only those rows are normed into ``out[r]`` and the streams are left as they are."""
+    _check(x, "x", torch.float32, 3)
+    T, n, H = x.shape
+    _check(out, "out", dims=2)
+    for t, name, shape in ((in_w, "in_w", (n,)), (weight, "weight", (H,)), (out_w, "out_w", (n,)), (mix, "mix", (n, n))):
+        if t is not None:
+            _check(t, name, torch.float32)
+            if tuple(t.shape) != shape:
+                raise KernelError(f"stream_norm: {name} {tuple(t.shape)} is not {shape}")
+    dptr, S, dstride = _delta(delta, T, H, "stream_norm")
+    if delta is not None and out_w is None:
+        raise KernelError("stream_norm: a pending result needs the streams' weights on it")
+    for t, name in ((slice_bias, "slice_bias"), (slice_weight, "slice_weight")):
+        if t is not None:
+            _check(t, name, torch.float32, 2)
+            if delta is None or tuple(t.shape) != (S, H):
+                raise KernelError(f"stream_norm: {name} must have one row per slice of the pending sums")
+    R = T
+    if rows is not None:
+        _check(rows, "rows", torch.int32, 1)
+        R = rows.shape[0]
+    if out.shape[0] < R or out.shape[1] != H:
+        raise KernelError("stream_norm: out has too few rows or another width")
+
+    def ptr(t):
+        return t.data_ptr() if t is not None else 0
+    call(core(), "ap_stream_norm", x.data_ptr(), ptr(rows), R, dptr, S, dstride, ptr(slice_bias), ptr(slice_weight),
+         float(slice_eps), float(slice_scale), ptr(out_w), ptr(mix), in_w.data_ptr(), weight.data_ptr(), float(eps),
+         0 if rows is not None else 1, out.data_ptr(), dtype_code(out.dtype), n, H, stream_handle())
 
 
 def bias_act(inp: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor, activation: Optional[str]) -> None:

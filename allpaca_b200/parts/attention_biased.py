@@ -17,10 +17,17 @@
 * ``output_gate``: head ``h`` of the result is multiplied by ``sigmoid(g h)_h``, one number per row and
   head from the mixer's input (tensor ``g [heads, hidden]``), before the output projection;
 * ``rope`` (a ``position`` part whose ``head_dim`` is the number of rotated coordinates): the first that many
-  coordinates of every normed query and key head are turned by the position, coordinate ``i`` with ``i + dims/2``,
-  the rest pass as they are;
+  coordinates of every normed query and key head are turned by the position, coordinate ``i`` with ``i + dims/2``
+  or, by the part's pairing, ``2i`` with ``2i + 1``; the rest pass as they are;
 * ``softcap`` ``c``: the scaled score becomes ``c * tanh(score / c)`` before bias and softmax;
-* ``qkv_bias``: Q, K and V have biases (tensors ``q.b``, ``k.b``, ``v.b``), added before the norm;
+* ``qkv_bias``: Q, K and V have biases (tensors ``q.b``, ``k.b``, ``v.b``), added before the norm; ``o_bias``: so
+  has the output projection (tensor ``o.b``);
+* ``conv_taps`` ``n > 0``: Q, K and V each pass a causal convolution over the last ``n`` tokens per channel (tensors
+  ``q.conv``, ``k.conv``, ``v.conv`` ``[channels, n]``, the last column on the row itself, zeros before the sequence's
+  start, no activation), after the bias and before norm and rotation; the last ``n - 1`` biased projections are
+  fixed-size state of the request, 32-bit;
+* ``sink``: the softmax's denominator also holds ``exp(sink[h])``, one learned number per query head (tensor
+  ``sink``) to which neither key nor value belongs;
 * ``output_scale``: the mixer's result times a constant (carried by the values on their way into the pages, so
   that it costs nothing).
 
@@ -45,9 +52,10 @@ class DistanceBiasedAttention(Mixer):
     """Parameters: ``hidden_size``, ``num_heads``, ``num_kv_heads``, ``head_dim``, ``value_dim``
     (None: ``head_dim``), ``scale``, ``window``, ``keep_first``, ``qk_norm_eps``, ``qk_norm_weights``,
     ``q_temp``, ``distance_bias``, ``slope_exponent``, ``output_gate``, ``rope``, ``softcap``, ``qkv_bias``,
-    ``output_scale``; tensors ``q``, ``k``, ``v``, ``o``
-    (``[out, in]``) and, by the parameters, ``r1``, ``r2`` (``[num_heads]``), ``q.norm``, ``k.norm``
-    (``[head_dim]``), ``g`` (``[num_heads, hidden]``)."""
+    ``o_bias``, ``conv_taps``, ``sink``, ``output_scale``; tensors ``q``, ``k``, ``v``, ``o``
+    (``[out, in]``) and, by the parameters, ``r1``, ``r2``, ``sink`` (``[num_heads]``), ``q.norm``, ``k.norm``
+    (``[head_dim]``), ``g`` (``[num_heads, hidden]``), ``q.b``, ``k.b``, ``v.b``, ``o.b``, ``q.conv``, ``k.conv``,
+    ``v.conv``."""
 
     MAX_HEAD = 256
 
@@ -90,12 +98,20 @@ class DistanceBiasedAttention(Mixer):
         self.o = Linear(env, self.hidden, self.nh * self.vd)
         self.r1 = self.r2 = self.q_weight = self.k_weight = self.qkv_bias = None
         self.position = build("position", p["rope"], env) if p.get("rope") is not None else None
-        if self.position is not None and (self.position.head_dim > self.hd or self.position.pairing != 0):
-            raise PartError(f"a rotation of {self.position.head_dim} coordinates in half-split pairs does not fit "
-                            f"heads of {self.hd}")
+        if self.position is not None and self.position.head_dim > self.hd:
+            raise PartError(f"a rotation of {self.position.head_dim} coordinates does not fit heads of {self.hd}")
         self.softcap = float(p["softcap"]) if p.get("softcap") else 0.0
         self.has_qkv_bias = bool(p.get("qkv_bias", False))
+        self.has_o_bias = bool(p.get("o_bias", False))
+        self.output_bias = None               # what `forward(..., add_bias=False)` leaves to its caller
+        self.taps = int(p.get("conv_taps") or 0)
+        self.conv_channels = self.q_size + self.k_size + self.v_size
+        self.conv_w = self.sink = None
+        self.has_sink = bool(p.get("sink", False))
         self.output_scale = float(p.get("output_scale", 1.0))
+
+    def state_bytes(self) -> int:
+        return 4 * max(self.taps - 1, 0) * self.conv_channels
 
     def parts(self):
         yield self
@@ -116,6 +132,14 @@ class DistanceBiasedAttention(Mixer):
         if self.has_qkv_bias:
             w.update({"q.b": WeightSpec((self.q_size,), "bias"), "k.b": WeightSpec((self.k_size,), "bias"),
                       "v.b": WeightSpec((self.v_size,), "bias")})
+        if self.has_o_bias:
+            w["o.b"] = WeightSpec((self.hidden,), "bias")
+        if self.taps > 0:
+            w.update({"q.conv": WeightSpec((self.q_size, self.taps), "bias"),
+                      "k.conv": WeightSpec((self.k_size, self.taps), "bias"),
+                      "v.conv": WeightSpec((self.v_size, self.taps), "bias")})
+        if self.has_sink:
+            w["sink"] = WeightSpec((self.nh,), "bias")
         return w
 
     def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
@@ -132,6 +156,12 @@ class DistanceBiasedAttention(Mixer):
                 .to(torch.float32).to(self.env.device)
         if self.has_qkv_bias:
             self.qkv_bias = torch.cat([tensors["q.b"], tensors["k.b"], tensors["v.b"]]).float().contiguous()
+        if self.has_o_bias:
+            self.output_bias = (tensors["o.b"].float() * self.output_scale).contiguous()
+        if self.taps > 0:
+            self.conv_w = torch.cat([tensors["q.conv"], tensors["k.conv"], tensors["v.conv"]], dim=0).float().contiguous()
+        if self.has_sink:
+            self.sink = tensors["sink"].float().contiguous()
         if self.qk_norm_weights:
             self.q_weight = tensors["q.norm"].float().contiguous()
             self.k_weight = tensors["k.norm"].float().contiguous()
@@ -140,12 +170,24 @@ class DistanceBiasedAttention(Mixer):
         return CacheNeed(outer=(self.nkv,), inner=(self.hd + self.vd,), window=self.window,
                          keep_first=self.keep_first)
 
-    def forward(self, h: torch.Tensor, step, cache: LayerCache, into=None) -> torch.Tensor:
+    def forward(self, h: torch.Tensor, step, cache: LayerCache, into=None, add_bias: bool = True) -> torch.Tensor:
         """``into`` (optional, 32-bit ``[T, hidden]``): where the output projection leaves its sums, for a mixer
-        that runs beside another one."""
+        that runs beside another one; ``add_bias`` False: the caller adds ``output_bias`` itself."""
         T = h.shape[0]
         ws = self.env.workspace
-        qkv = self.qkv.forward(h, "battn.qkv", "float32")
+        proj = qkv = self.qkv.forward(h, "battn.qkv", "float32")
+        bias = self.qkv_bias
+        if self.taps > 0:
+            conv_state = None
+            if self.taps > 1:
+                if cache.state is None:
+                    raise PartError("attention behind a convolution needs a state slot per request")
+                conv_state = cache.state.view(torch.float32)[:, :(self.taps - 1) * self.conv_channels] \
+                    .unflatten(1, (self.taps - 1, self.conv_channels))
+            qkv = ws.get("battn.conv", (T, self.conv_channels), torch.float32)
+            ops.causal_conv(proj, 0, self.conv_w, None, conv_state, step.seq_start, step.positions, step.state_slots,
+                            qkv, step.num_seqs, activation=None, in_bias=bias)
+            bias = None
         cos_sin = self.position.rotation_for(step)[0] if self.position is not None else None
         q = ws.get("battn.q", (T, self.q_size), self.env.dtype)
         table = step.block_tables[cache.group]
@@ -153,8 +195,10 @@ class DistanceBiasedAttention(Mixer):
                           self.nh, self.nkv, self.hd, self.vd, self.qk_norm_eps or 0.0,
                           normalise=self.qk_norm_eps is not None, temp_coef=self.temp_coef,
                           temp_every=self.temp_every, q_weight=self.q_weight, k_weight=self.k_weight,
-                          bias=self.qkv_bias, cos_sin=cos_sin, value_scale=self.output_scale)
-        gate = qkv[:, self.q_size + self.k_size + self.v_size:] if self.output_gate else None
+                          bias=bias, cos_sin=cos_sin,
+                          pairing=self.position.pairing if self.position is not None else 0,
+                          value_scale=self.output_scale)
+        gate = proj[:, self.q_size + self.k_size + self.v_size:] if self.output_gate else None
         out = ws.get("battn.out", (T, self.nh * self.vd), self.env.dtype)
         # bfloat16: one-row sequences on the decode kernel (a step of such rows only is what a CUDA graph
         # records, and every replay is again such a step); 32-bit: one kernel for all rows, so that a
@@ -164,6 +208,9 @@ class DistanceBiasedAttention(Mixer):
         ops.attention_window_bias(q, out, cache.pages, table, step.seq_start, step.positions, step.num_seqs,
                                   self.nh, self.nkv, self.hd, self.vd, self.scale, self.window or 0, self.r1, self.r2,
                                   single_rows=single, other_rows=step.max_query_len != 1, bias=self.bias_kind,
-                                  keep_first=self.keep_first, gate=gate, softcap=self.softcap,
+                                  keep_first=self.keep_first, gate=gate, softcap=self.softcap, sink=self.sink,
                                   max_context=step.max_decode_context_len or step.max_context_len)
-        return self.o.forward(out, "battn.o", "delta", into=into)
+        delta = self.o.forward(out, "battn.o", "delta", into=into)
+        if self.output_bias is not None and add_bias:
+            ops.bias_add(delta if into is not None else delta[0], self.output_bias)
+        return delta

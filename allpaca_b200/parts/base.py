@@ -13,7 +13,8 @@ Kinds of part and what each must provide
 ``position``      :class:`PositionEncoding`  injects positions into queries and keys
 ``block``         :class:`Block`        arranges the parts above around the residual stream
 ``stream``        :class:`Part`         acts on the residual stream around a layer's sublayers (a mix with
-                                        the previous token's row, an average over the layers' results)
+                                        the previous token's row, an average over the layers' results, weights
+                                        between several streams and a sublayer)
 
 All parts share :class:`Part`: ``weights()`` names the tensors they need (local
 names, shapes, roles) and ``load()`` receives them.  A part is registered with
@@ -188,6 +189,29 @@ class Deferred:
     parts: int
 
 
+@dataclass
+class Slices:
+    """A sublayer's unfinished result: 32-bit sums ``[S, T, hidden]`` whose finish is left to whoever adds them to the
+    residual.  ``bias [S, hidden]`` (None: none) belongs to the sums; with ``weight [S, hidden]`` every slice is divided
+    by its own root mean square (``eps``), multiplied by its weight and by ``scale``; the result is the slices' sum."""
+
+    sums: torch.Tensor
+    bias: Optional[torch.Tensor] = None
+    weight: Optional[torch.Tensor] = None
+    eps: float = 0.0
+    scale: float = 1.0
+
+
+@dataclass
+class StreamUpdate:
+    """What a block with several residual streams hands on: its last sublayer's result and how the streams take it,
+    ``x_t <- sum_s mix[s, t] x_s + out_w[t] y`` (``mix`` None: the old streams do not enter)."""
+
+    result: Slices
+    out_w: torch.Tensor
+    mix: Optional[torch.Tensor] = None
+
+
 class Part:
     """Common face of every part."""
 
@@ -232,6 +256,11 @@ class Norm(Part):
         """For blocks that norm a sublayer's output instead of its input: add ``mult`` times the
         normalised ``delta`` (32-bit partial sums) into the residual ``x``; ``copy`` (optional)
         receives the updated rows in its own type."""
+        raise NotImplementedError
+
+    def forward_streams(self, x, in_w, out, pending=None, rows=None) -> None:
+        """For residuals of several streams ``x [T, n, hidden]``: apply ``pending`` (:class:`StreamUpdate` or None),
+        then norm ``sum_s in_w[s] x_s``.  With ``rows`` only those rows are produced and ``x`` is left untouched."""
         raise NotImplementedError
 
 
@@ -332,6 +361,9 @@ class ModelSpec:
     head_name: str = "lm_head.weight"
     tie_word_embeddings: bool = False
     max_position_embeddings: int = 2048
+    # The residual is this many streams ``[T, streams, hidden]`` that start as copies of the embedding row and are
+    # summed at the end (None: one vector); every block must then be one that keeps streams.
+    streams: Optional[int] = None
     # Ends of the stack that some decoders alter; all default to "as it is".
     embedding_scale: Optional[float] = None      # the gathered embedding row is multiplied by it
     # sinusoidal position vector added to the embedding row: with angle a_i = p * base^(-2i/width), column 2i

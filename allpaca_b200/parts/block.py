@@ -13,7 +13,8 @@ from typing import Dict
 import torch
 
 from .. import ops
-from .base import Block, BuildEnv, Deferred, LayerCache, Part, PartError, build, register
+from .base import (Block, BuildEnv, Deferred, LayerCache, Part, PartError, Slices, StreamUpdate, build,
+                   register)
 from .norm import RMSNorm
 
 
@@ -261,6 +262,61 @@ class GatedPostNormBlock(Block):
             self._sublayer(x, h, copy, self.feed_forward, self.feed_forward_gate, self.feed_forward_norm, step)
         step.shared["block.stream_copy"] = x     # the copy is up to date with this residual
         return None
+
+
+@register("block", "hyper_connections")
+class HyperConnectionsBlock(Block):
+    """A pre-norm layer on a residual of several streams ``x [T, n, hidden]``:
+
+    ``u = sum_s in[s] x_s``;  ``y = sublayer(norm(u))``;  ``x_t <- sum_s mix[s, t] x_s + out[t] y``
+
+    for the mixer and again, with weights of its own, for the feed-forward.  A sublayer's result is applied by the
+    norm that reads the streams next (in the layer or the one after), in one kernel; the block hands its last one on
+    as a :class:`StreamUpdate`.  A mixer that offers ``forward_slices`` leaves the finish of its result to that kernel.
+
+    Parameters: ``hidden_size``, ``streams``, ``mixer``, ``feed_forward`` (None: the mixer alone), ``mixer_norm``,
+    ``feed_forward_norm`` (norms that offer ``forward_streams``), ``mixer_streams``, ``feed_forward_streams``
+    (``stream`` parts with ``in_w``, ``out_w``, ``mix``), and the weight-name prefixes of :class:`PreNormBlock` plus
+    ``mixer_streams_prefix``, ``feed_forward_streams_prefix``."""
+
+    def __init__(self, params, env: BuildEnv):
+        super().__init__(params, env)
+        self.require("hidden_size", "streams", "mixer", "mixer_norm", "mixer_streams")
+        self.hidden, self.streams = int(params["hidden_size"]), int(params["streams"])
+        self.feed_forward = self.feed_forward_norm = self.feed_forward_streams = None
+        self._prefixes = {}
+
+        def part(kind, name, prefix):
+            made = build(kind, params[name], env)
+            self._prefixes[params.get(name + "_prefix", prefix)] = made
+            return made
+        self.mixer = part("mixer", "mixer", "mixer.")
+        self.mixer_norm = part("norm", "mixer_norm", "mixer_norm.")
+        self.mixer_streams = part("stream", "mixer_streams", "mixer_streams.")
+        if params.get("feed_forward") is not None:
+            self.require("feed_forward_norm", "feed_forward_streams")
+            self.feed_forward = part("feed_forward", "feed_forward", "feed_forward.")
+            self.feed_forward_norm = part("norm", "feed_forward_norm", "feed_forward_norm.")
+            self.feed_forward_streams = part("stream", "feed_forward_streams", "feed_forward_streams.")
+
+    def sub_parts(self) -> Dict[str, Part]:
+        return dict(self._prefixes)
+
+    def _sublayer(self, x, pending, norm, weights, run) -> StreamUpdate:
+        h = self.env.workspace.get("block.normed", (x.shape[0], self.hidden), self.env.dtype)
+        norm.forward_streams(x, weights.in_w, h, pending=pending)
+        y = run(h)
+        return StreamUpdate(y if isinstance(y, Slices) else Slices(y), weights.out_w, weights.mix)
+
+    def forward(self, x: torch.Tensor, delta, step, cache: LayerCache):
+        if x.dim() != 3 or x.shape[1] != self.streams or not (delta is None or isinstance(delta, StreamUpdate)):
+            raise PartError(f"this block keeps {self.streams} residual streams; the model's residual is {tuple(x.shape)}")
+        mix = getattr(self.mixer, "forward_slices", self.mixer.forward)
+        delta = self._sublayer(x, delta, self.mixer_norm, self.mixer_streams, lambda h: mix(h, step, cache))
+        if self.feed_forward is not None:
+            delta = self._sublayer(x, delta, self.feed_forward_norm, self.feed_forward_streams,
+                                   lambda h: self.feed_forward.forward(h, step))
+        return delta
 
 
 class _Several(Part):

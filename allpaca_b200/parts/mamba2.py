@@ -88,8 +88,8 @@ class Mamba2(Mixer):
         conv_state = rows[:, self.ssm_floats:].unflatten(1, (self.taps - 1, self.conv_channels)) \
             if self.taps > 1 else None
         xbc = ws.get("mamba.xbc", (T, self.conv_channels), torch.float32)
-        ops.causal_conv_silu(proj, self.inner, self.conv_w, self.conv_b, conv_state, step.token_seq, step.seq_start,
-                             step.positions, step.state_slots, xbc, S)
+        ops.causal_conv(proj, self.inner, self.conv_w, self.conv_b, conv_state, step.seq_start, step.positions,
+                        step.state_slots, xbc, S)
         y = ws.get("mamba.y", (T, self.inner), torch.float32)
         ops.ssm_scan(xbc, proj[:, self.inner + self.conv_channels:], self.dt_bias, self.a_log, self.d_skip,
                      ssm_state, step.seq_start, step.positions, step.state_slots, y, S, self.heads, self.groups,

@@ -19,7 +19,8 @@ class RMSNorm(Norm):
     """Parameters: ``size`` (width of a row), ``eps``, ``scalar_weight`` (False; True: the
     checkpoint holds one number for all coordinates, a tensor without dimensions), ``weight_name``
     (``"weight"``: the tensor's name behind the part's prefix; may be empty, the prefix then is
-    the whole name)."""
+    the whole name), ``weight_offset`` (0; 1: the weight is stored around zero and counts as ``1 + w``,
+    formed in 32-bit)."""
 
     def __init__(self, params, env: BuildEnv):
         super().__init__(params, env)
@@ -28,17 +29,22 @@ class RMSNorm(Norm):
         self.eps = float(params["eps"])
         self.scalar_weight = bool(params.get("scalar_weight", False))
         self.weight_name = str(params.get("weight_name", "weight"))
+        self.weight_offset = float(params.get("weight_offset", 0.0))
         self.weight = None
-        self._kernel_weight = None
+        self._kernel_weight = self._weight32 = None
 
     def weights(self) -> Dict[str, WeightSpec]:
-        return {self.weight_name: WeightSpec(() if self.scalar_weight else (self.size,), "norm")}
+        # a weight stored around zero is drawn like a bias where weights are random
+        return {self.weight_name: WeightSpec(() if self.scalar_weight else (self.size,),
+                                             "norm" if self.weight_offset == 0.0 else "bias")}
 
     def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
         w = tensors[self.weight_name]
+        if self.weight_offset != 0.0:
+            w = w.float() + self.weight_offset
         # one number for all coordinates: the kernels take it as a vector of equal entries
         self.weight = (w.reshape(1).expand(self.size) if self.scalar_weight else w).contiguous()
-        self._kernel_weight = self.weight
+        self._kernel_weight, self._weight32 = self.weight, None
 
     def fold(self) -> None:
         """The weight has been multiplied into the product that consumes this norm's output:
@@ -56,6 +62,16 @@ class RMSNorm(Norm):
         """The norm on a sublayer's output: ``x += mult * norm(delta)``; ``copy`` (optional) receives
         the updated rows in its own type."""
         ops.norm_residual(x, delta, self.weight, self.eps, mult, copy)
+
+    def forward_streams(self, x, in_w, out, pending=None, rows=None) -> None:
+        if self._weight32 is None:
+            self._weight32 = self._kernel_weight.float().contiguous()
+        if pending is None:
+            ops.stream_norm(x, in_w, self._weight32, self.eps, out, rows=rows)
+            return
+        y = pending.result
+        ops.stream_norm(x, in_w, self._weight32, self.eps, out, delta=y.sums, out_w=pending.out_w, mix=pending.mix,
+                        slice_bias=y.bias, slice_weight=y.weight, slice_eps=y.eps, slice_scale=y.scale, rows=rows)
 
 
 @register("norm", "dynamic_tanh")

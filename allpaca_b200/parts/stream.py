@@ -11,6 +11,9 @@ output.  The results of a step's rows wait in a workspace buffer ``[count, T, hi
 kept between steps.  All 32-bit.
 
 ``residual_gate``: a gate per coordinate on what a sublayer adds to the stream, read off the sublayer's input.
+
+``stream_weights``: where the residual is several streams, how one sublayer reads them, writes them and lets them
+mix; the arithmetic lives in the norm before the next sublayer (``forward_streams``).
 """
 from __future__ import annotations
 
@@ -106,3 +109,27 @@ class ResidualGate(Part):
     def forward(self, h: torch.Tensor) -> torch.Tensor:
         """The gate's logits without the bias, 32-bit ``[T, hidden]``."""
         return self.linear.forward(h, "stream.gate." + self.name, "float32")
+
+
+@register("stream", "stream_weights")
+class StreamWeights(Part):
+    """One sublayer's weights between ``streams`` residual streams and itself: it reads ``sum_s in_w[s] x_s``; its
+    result goes back as ``x_t <- sum_s mix[s, t] x_s + out_w[t] y``.  32-bit in both engine types.
+
+    Parameters: ``streams``, ``names`` (tensor names of the three, default ``("in", "out", "mix")``; ``mix`` is indexed
+    [from, to])."""
+
+    def __init__(self, params, env: BuildEnv):
+        super().__init__(params, env)
+        self.require("streams")
+        self.streams = int(params["streams"])
+        self.names = tuple(params.get("names") or ("in", "out", "mix"))
+        self.in_w = self.out_w = self.mix = None
+
+    def weights(self) -> Dict[str, WeightSpec]:
+        n = self.streams
+        return {self.names[0]: WeightSpec((n,), "norm"), self.names[1]: WeightSpec((n,), "norm"),
+                self.names[2]: WeightSpec((n, n), "bias")}
+
+    def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
+        self.in_w, self.out_w, self.mix = (tensors[n].float().contiguous() for n in self.names)

@@ -140,14 +140,14 @@ def test_query_and_key_norm_temperature_and_store(dtype):
         close(slot[:, D:], qkv[i, (H + G) * D:].view(G, E), tol, ("value", p))
 
 
-@pytest.mark.parametrize("taps,C", [(4, 37), (2, 64), (3, 300), (1, 5)])
+@pytest.mark.parametrize("taps,C", [(4, 37), (2, 64), (3, 300), (1, 5), (5, 8), (6, 12), (7, 12), (12, 20)])
 def test_convolution_carried_over_portions(taps, C):
     """Two sequences in alternating slots, cut into portions of 1, 2, 1, 5, 3 ... rows (shorter than
     the convolution), each step one launch over both."""
     from allpaca_b200 import ops
     g = torch.Generator().manual_seed(taps)
     L = [23, 17]
-    u = [torch.randn(n, C + 6, generator=g) for n in L]
+    u = [torch.randn(n, C + 8, generator=g) for n in L]
     w, b = torch.randn(C, taps, generator=g), torch.randn(C, generator=g)
     want = [plain.silu(plain.causal_conv(x[:, 4:4 + C].double(), w.double(), b.double())) for x in u]
     state = torch.full((3, max(taps - 1, 1), C), float("nan"), device=DEV)      # slots 2 and 0 are used
@@ -169,10 +169,9 @@ def test_convolution_carried_over_portions(taps, C):
         for _, _, n in seqs:
             starts.append(starts[-1] + n)
         out = torch.empty(T, C, device=DEV)
-        ops.causal_conv_silu(x, 4, w.to(DEV), b.to(DEV), state if taps > 1 else None,
-                             i32([j for j, (_, _, n) in enumerate(seqs) for _ in range(n)]), i32(starts),
-                             i32([a + i for _, a, n in seqs for i in range(n)]), i32([2 if s == 0 else 0 for s, _, _ in seqs]),
-                             out, len(seqs))
+        ops.causal_conv(x, 4, w.to(DEV), b.to(DEV), state if taps > 1 else None, i32(starts),
+                        i32([a + i for _, a, n in seqs for i in range(n)]), i32([2 if s == 0 else 0 for s, _, _ in seqs]),
+                        out, len(seqs))
         for j, (s, a, n) in enumerate(seqs):
             got[s].append(out[starts[j]:starts[j + 1]].cpu())
             at[s] += n

@@ -1,9 +1,10 @@
 """Prefill and decode throughput of one design beside the dense Llama decoder of equal size,
 with the time of every kind of kernel in a step:
 
-    python bench.py --design viresun|bivatar|lazolix|gezozen [--design-size small|base|wide]
+    python bench.py --design viresun|bivatar|lazolix|gezozen|boketar [--design-size small|base|wide]
 
-Gezozen runs beside the Viresun decoder (the closest existing model: windowed attention, a recurrent mixer
+Boketar runs beside the Gezozen decoder (the closest existing model: softmax attention beside a linear attention, a
+delta rule with short convolutions) and the Llama decoder.  Gezozen runs beside the Viresun decoder (the closest existing model: windowed attention, a recurrent mixer
 with fixed-size state, routed experts) and the Llama decoder.  Lazolix runs beside two models: the Bivatar decoder reduced to its latent layers (the closest existing
 mixer) and the Llama decoder.  All models have random bfloat16 weights drawn on the device, the same width, heads, head size,
 feed-forward size, number of layers and vocabulary.  Timed on the device with CUDA events after
@@ -108,6 +109,27 @@ def gezozen_config(size: str) -> dict:
                        {"type": "parallel_2", "mixer": pair2, "mlp": moe}, {"type": "delta", "mixer": delta, "mlp": moe}]}
 
 
+STREAMS = 4                     # residual streams of the Boketar decoder
+NARROW = 128                    # inner width of its narrow pairs of products
+
+
+def boketar_config(size: str) -> dict:
+    """Four layers with dense feed-forwards on four residual streams: a delta rule with a decay per key channel;
+    windowed attention with short convolutions and a sink beside lightning attention; the same two again."""
+    W, H, G, D, ff = SIZES[size][:5]
+    window = SIZES[size][8]
+    delta = {"heads": H, "kv_heads": G, "dim": D, "vdim": D, "conv": 4, "decay_rank": NARROW, "gate_rank": NARROW}
+    half = max(H // 2, 1)
+    pair = {"left": {"heads": H, "kv_heads": G, "dim": D, "vdim": D, "scale": D ** -0.5, "mask": {"size": window},
+                     "rot": {"base": 10000.0, "dims": D // 2}, "conv": 3},
+            "right": {"heads": half, "dim": D, "vdim": D, "decay": [1.0 - 2.0 ** (-5 - (i % 6)) for i in range(half)]}}
+    dense = {"kind": "dense", "ff": ff}
+    return {"architecture": "Boketar", "vocab": VOCAB, "width": W, "norm": {"eps": 1e-6}, "streams": STREAMS,
+            "embedding": {"scale": 8.0},
+            "layers": [{"type": "channel_delta", "mixer": delta, "mlp": dense}, {"type": "parallel", "mixer": pair, "mlp": dense},
+                       {"type": "channel_delta", "mixer": delta, "mlp": dense}, {"type": "parallel", "mixer": pair, "mlp": dense}]}
+
+
 def bivatar_latent_config(size: str) -> dict:
     """The Bivatar decoder with latent layers only (the windowed layer left out): what Lazolix runs beside."""
     raw = bivatar_config(size)
@@ -119,6 +141,9 @@ def bivatar_latent_config(size: str) -> dict:
 
 
 DESIGNS = {
+    "boketar": (boketar_config, "hyper-connections over 4 residual streams; delta rule with a decay per key channel, "
+                                "windowed attention with short convolutions and a sink beside lightning attention, "
+                                "the same two again; dense feed-forwards"),
     "gezozen": (gezozen_config, "norm after the gated sum; gated delta rule, softmax attention beside gated linear "
                                 "attention, windowed softmax attention beside retention, gated delta rule; routed "
                                 "experts with a gated shared expert in every layer"),
@@ -269,6 +294,10 @@ def run(design: str, size: str, steps: int, warmup: int, batch: int, context: in
         R, _, nope, _, vd, _ = LATENT_SIZES[size]
         sizes.update({"kv_rank": R, "dim": nope, "vdim": vd, "identity": 2})
         others.insert(0, ("bivatar_latent", bivatar_latent_config(size)))
+    if design == "boketar":
+        sizes = {k: v for k, v in sizes.items() if k in ("width", "heads", "kv_heads", "head_dim", "ff", "window")}
+        sizes.update({"lightning_heads": max(sizes["heads"] // 2, 1), "streams": STREAMS, "narrow": NARROW})
+        others.insert(0, ("gezozen", gezozen_config(size)))
     if design == "gezozen":
         sizes = {k: v for k, v in sizes.items() if k in ("width", "heads", "kv_heads", "head_dim", "experts", "top",
                                                          "expert_ff", "window")}

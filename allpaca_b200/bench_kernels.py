@@ -435,10 +435,13 @@ def bench_stream(args) -> dict:
 
 
 def bench_recurrent(args) -> dict:
-    """The linear-attention recurrence in its three kinds (a decay per channel; a fixed decay per head with rotated
-    queries and keys; the gated delta rule with unit vectors) on ``--seqs`` sequences of ``--rows`` rows each, beside
+    """The linear-attention recurrence in its kinds (a decay per channel; a fixed decay per head with rotated
+    queries and keys, or with SiLU on queries, keys and values; the gated delta rule with unit vectors, with a decay
+    per head and with one per channel) on ``--seqs`` sequences of ``--rows`` rows each, beside
     the state-space recurrence of the same state size (``ssm_scan``); and the norm after a gated sum beside
-    ``add_rmsnorm`` and ``norm_residual`` on the same rows, each beside the bytes it must move."""
+    ``add_rmsnorm`` and ``norm_residual`` on the same rows, the norm behind hyper-connections of ``--streams`` residual
+    streams (with one pending slice, and with two that are normed on their own), and the causal convolution, each
+    beside the bytes it must move."""
     from allpaca_b200 import ops
     n, S, H, D, V, W = args.rows, max(1, args.seqs), args.heads, args.dim, args.vdim, args.width
     T = n * S
@@ -456,22 +459,28 @@ def bench_recurrent(args) -> dict:
     seq_start = torch.arange(0, T + 1, n, dtype=torch.int32, device=dev)
     positions = torch.cat([torch.arange(7, 7 + n, dtype=torch.int32) for _ in range(S)]).to(dev)
     slots = torch.arange(S, dtype=torch.int32, device=dev)
-    token_seq = torch.arange(S, dtype=torch.int32, device=dev).repeat_interleave(n)
     consts = torch.full((H,), 0.99, device=dev)
-    a_log, dt_bias = torch.log(0.05 + 0.5 * torch.rand(H, device=dev)), rnd(H)
+    a_log, dt_bias, dt_channel = torch.log(0.05 + 0.5 * torch.rand(H, device=dev)), rnd(H), rnd(H * D)
     table = torch.empty(T, D // 2, 2, device=dev)
     ops.rope_table(positions, torch.pow(10000.0, -torch.arange(D // 2, device=dev) / (D // 2)).float(), table, 1.0)
+    from allpaca_b200.parts import Workspace
+    ws = None if args.token_by_token else Workspace(torch.device(dev))
     common = (y, state, seq_start, positions, slots, S, H, H, D, V)
     io = T * (2 * H * D + 2 * H * V) * 4 + 2 * S * H * D * V * 4
     cases = {
         "la_scan channel": (lambda i: ops.linear_scan(q[i % copies], k[i % copies], v[i % copies], *common, "channel",
-                                                      decay_channel=z[i % copies], tau=16.0, out_scale=D ** -0.5),
+                                                      workspace=ws, decay_channel=z[i % copies], tau=16.0, out_scale=D ** -0.5),
                             io + T * H * D * 4),
         "la_scan head, rotated": (lambda i: ops.linear_scan(q[i % copies], k[i % copies], v[i % copies], *common, "head",
-                                                            decay_const=consts, qk="rotate", cos_sin=table), io),
+                                                            workspace=ws, decay_const=consts, qk="rotate", cos_sin=table), io),
         "la_scan delta rule": (lambda i: ops.linear_scan(q[i % copies], k[i % copies], v[i % copies], *common,
-                                                         "head_token", decay_head=a, decay_const=a_log, dt_bias=dt_bias,
+                                                         "head_token", workspace=ws, decay_head=a, decay_const=a_log, dt_bias=dt_bias,
                                                          beta=b, qk="unit", unit_eps=1e-6), io),
+        "la_scan head, silu": (lambda i: ops.linear_scan(q[i % copies], k[i % copies], v[i % copies], *common, "head",
+                                                         workspace=ws, decay_const=consts, qk="silu"), io),
+        "la_scan channel delta rule": (lambda i: ops.linear_scan(
+            q[i % copies], k[i % copies], v[i % copies], *common, "channel_token", workspace=ws, decay_channel=z[i % copies],
+            decay_const=a_log, dt_bias=dt_channel, beta=b, qk="unit", unit_eps=1e-6), io + T * H * D * 4),
     }
     # the state-space recurrence with the same state per head: B and C of D numbers, one group per head
     xbc = [rnd(T, H * V + 2 * H * D) for _ in range(copies)]
@@ -495,6 +504,23 @@ def bench_recurrent(args) -> dict:
     cases["norm_residual"] = (lambda i: ops.norm_residual(xs[i % wc], ds[i % wc], w32, 1e-6, 0.5, copy), T * W * 14)
     cases["add_rmsnorm"] = (lambda i: ops.add_rmsnorm(xs[i % wc], w32.to(torch.bfloat16), 1e-6, copy, delta=ds[i % wc]),
                             T * W * 14)
+    N = args.streams
+    sc = max(2, int(math.ceil(300e6 / (T * W * N * 4))))
+    streams = [rnd(T, N, W) for _ in range(sc)]
+    pend, pend2 = [rnd(1, T, W) for _ in range(sc)], [rnd(2, T, W) for _ in range(sc)]
+    win, wout, wmix = torch.full((N,), 1.0 / N, device=dev), torch.ones(N, device=dev), torch.eye(N, device=dev)
+    sb, sw = rnd(2, W), torch.ones(2, W, device=dev)
+    cases[f"stream_norm, {N} streams"] = (lambda i: ops.stream_norm(streams[i % sc], win, w32, 1e-6, copy, delta=pend[i % sc],
+                                                                   out_w=wout, mix=wmix), T * W * (8 * N + 6))
+    cases[f"stream_norm, {N} streams, two normed slices"] = (
+        lambda i: ops.stream_norm(streams[i % sc], win, w32, 1e-6, copy, delta=pend2[i % sc], out_w=wout, mix=wmix,
+                                  slice_bias=sb, slice_weight=sw, slice_eps=1e-6), T * W * (8 * N + 10))
+    C = 2 * H * D + H * V
+    cc = max(2, int(math.ceil(300e6 / (T * C * 4))))
+    cin = [rnd(T, C) for _ in range(cc)]
+    conv_out, conv_w, conv_state = torch.empty(T, C, device=dev), rnd(C, 4), torch.zeros(S, 3, C, device=dev)
+    cases["causal_conv, 4 taps"] = (lambda i: ops.causal_conv(cin[i % cc], 0, conv_w, None, conv_state, seq_start, positions,
+                                                              slots, conv_out, S), T * C * 8 + S * C * 24)
     res = {"rows_per_seq": n, "seqs": S, "heads": H, "dim": D, "vdim": V, "width": W, "groups": args.groups}
     for name, (fn, nbytes) in cases.items():
         us = _time(fn, args.iters, args.warmup, not args.no_graph)
@@ -617,6 +643,8 @@ def main(argv=None) -> int:
     s.add_argument("--vdim", type=int, default=128)
     s.add_argument("--width", type=int, default=2048)
     s.add_argument("--groups", type=int, default=4)
+    s.add_argument("--streams", type=int, default=4)
+    s.add_argument("--token-by-token", action="store_true", help="never eight tokens at a time")
     s = sub.add_parser("versus-reference")
     s.add_argument("--iters", type=int, default=20)
     s.add_argument("--warmup", type=int, default=3)

@@ -58,12 +58,32 @@ template <int VEC> __device__ __forceinline__ void hc_store(bf16* p, const float
     }
 }
 
-// NS: the number of streams the kernel is built for (0: any number up to HC_MAX_STREAMS)
-template <int NS, int VEC, typename TO>
-__global__ void stream_norm_kernel(const StreamNormArgs A, TO* __restrict__ out) {
+// sums over the CTA of up to HC_MAX_SLICES numbers a thread, in a fixed order, between two barriers
+__device__ __forceinline__ void hc_block_sums(float (&v)[HC_MAX_SLICES], int count, float (*scratch)[32]) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = (blockDim.x + 31) >> 5;
+#pragma unroll
+    for (int s = 0; s < HC_MAX_SLICES; ++s)
+        if (s < count) {
+            v[s] = ap_warp_sum(v[s]);
+            if (lane == 0) scratch[s][warp] = v[s];
+        }
+    __syncthreads();
+#pragma unroll
+    for (int s = 0; s < HC_MAX_SLICES; ++s)
+        if (s < count) {
+            float total = 0.f;
+            for (int w = 0; w < nwarps; ++w) total += scratch[s][w];
+            v[s] = total;
+        }
+}
+
+// NS: the number of streams the kernel is built for (0: any number up to HC_MAX_STREAMS).  ONE: the CTA has a thread for
+// every VEC columns, whose numbers stay in registers between the sums over the row.
+template <int NS, int VEC, bool ONE, typename TO>
+__global__ void __launch_bounds__(ONE && NS <= 4 ? 1024 : 512) stream_norm_kernel(const StreamNormArgs A, TO* __restrict__ out) {
     constexpr int N = NS ? NS : HC_MAX_STREAMS;
-    extern __shared__ __align__(16) float u_s[];             // [H]
-    __shared__ float scratch[32];
+    extern __shared__ __align__(16) float u_s[];             // [H] where not ONE
+    __shared__ float slice_scratch[HC_MAX_SLICES][32], scratch[32];
     __shared__ float mix_s[N * N], out_s[N], in_s[N];
     const int n = NS ? NS : A.streams;
     ap_pdl_trigger();
@@ -79,66 +99,58 @@ __global__ void stream_norm_kernel(const StreamNormArgs A, TO* __restrict__ out)
     float* xr = A.x + t * n * H;
     const float* dr = A.delta ? A.delta + t * H : nullptr;
     const bool reads_old = A.delta == nullptr || A.mix != nullptr;
-    float factor[HC_MAX_SLICES];
-#pragma unroll
-    for (int s = 0; s < HC_MAX_SLICES; ++s) factor[s] = 1.0f;
-    if (dr && A.slice_w) {
-#pragma unroll
-        for (int s = 0; s < HC_MAX_SLICES; ++s) {
-            if (s >= A.S) break;
-            float ss = 0.f;
-            for (int c = threadIdx.x * VEC; c < H; c += blockDim.x * VEC) {
-                float d[VEC], b[VEC];
-                hc_load<VEC>(dr + s * A.slice_stride + c, d);
-                if (A.slice_bias) {
-                    hc_load<VEC>(A.slice_bias + (size_t)s * H + c, b);
-#pragma unroll
-                    for (int i = 0; i < VEC; ++i) d[i] += b[i];
-                }
-#pragma unroll
-                for (int i = 0; i < VEC; ++i) ss = fmaf(d[i], d[i], ss);
-            }
-            ss = ap_block_sum(ss, scratch);
-            factor[s] = A.slice_scale / sqrtf(ss / (float)H + A.slice_eps);
-        }
-    }
-    __syncthreads();                                         // the weights are in shared memory
-    float ss = 0.f;
-    for (int c = threadIdx.x * VEC; c < H; c += blockDim.x * VEC) {
-        float old[N][VEC], u[VEC];
+    const bool normed = dr != nullptr && A.slice_w != nullptr;
+
+    auto load_old = [&](int c, float (&old)[N][VEC]) {
         if (reads_old) {
 #pragma unroll(NS ? N : 1)
-            for (int s = 0; s < N; ++s)
-                if (s < n) hc_load<VEC>(xr + (size_t)s * H + c, old[s]);
+            for (int s = 0; s < N; ++s) {
+                if (s >= n) break;
+                hc_load<VEC>(xr + (size_t)s * H + c, old[s]);
+            }
         }
+    };
+    auto load_slice = [&](int s, int c, float (&d)[VEC]) {
+        hc_load<VEC>(dr + s * A.slice_stride + c, d);
+        if (A.slice_bias) {
+            float b[VEC];
+            hc_load<VEC>(A.slice_bias + (size_t)s * H + c, b);
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) d[i] += b[i];
+        }
+    };
+    float factor[HC_MAX_SLICES];
+#pragma unroll
+    for (int s = 0; s < HC_MAX_SLICES; ++s) factor[s] = 0.f;
+    auto square = [&](int s, const float (&d)[VEC]) {
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) factor[s] = fmaf(d[i], d[i], factor[s]);
+    };
+    auto finish_factors = [&]() {
+        hc_block_sums(factor, A.S, slice_scratch);
+#pragma unroll
+        for (int s = 0; s < HC_MAX_SLICES; ++s) factor[s] = A.slice_scale / sqrtf(factor[s] / (float)H + A.slice_eps);
+    };
+    auto add_slice = [&](int s, int c, const float (&d)[VEC], float (&y)[VEC]) {
+        if (normed) {
+            float w[VEC];
+            hc_load<VEC>(A.slice_w + (size_t)s * H + c, w);
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) y[i] += d[i] * factor[s] * w[i];
+        } else {
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) y[i] += d[i];
+        }
+    };
+    // the streams after the pending result, and what the next sublayer reads of them
+    auto apply = [&](int c, const float (&old)[N][VEC], const float (&y)[VEC], float (&u)[VEC]) {
 #pragma unroll
         for (int i = 0; i < VEC; ++i) u[i] = 0.f;
-        if (dr) {
-            float y[VEC];
-#pragma unroll
-            for (int i = 0; i < VEC; ++i) y[i] = 0.f;
-#pragma unroll
-            for (int s = 0; s < HC_MAX_SLICES; ++s) {
-                if (s >= A.S) break;
-                float d[VEC], b[VEC];
-                hc_load<VEC>(dr + s * A.slice_stride + c, d);
-                if (A.slice_bias) {
-                    hc_load<VEC>(A.slice_bias + (size_t)s * H + c, b);
-#pragma unroll
-                    for (int i = 0; i < VEC; ++i) d[i] += b[i];
-                }
-                if (A.slice_w) {
-                    hc_load<VEC>(A.slice_w + (size_t)s * H + c, b);
-#pragma unroll
-                    for (int i = 0; i < VEC; ++i) d[i] = d[i] * factor[s] * b[i];
-                }
-#pragma unroll
-                for (int i = 0; i < VEC; ++i) y[i] += d[i];
-            }
 #pragma unroll(NS ? N : 1)
-            for (int o = 0; o < N; ++o) {
-                if (o >= n) break;
-                float v[VEC];
+        for (int o = 0; o < N; ++o) {
+            if (o >= n) break;
+            float v[VEC];
+            if (dr) {
 #pragma unroll
                 for (int i = 0; i < VEC; ++i) v[i] = out_s[o] * y[i];
                 if (A.mix) {
@@ -151,33 +163,94 @@ __global__ void stream_norm_kernel(const StreamNormArgs A, TO* __restrict__ out)
                     }
                 }
                 if (A.update) hc_store<VEC>(xr + (size_t)o * H + c, v);
-                const float wi = in_s[o];
+            } else {
 #pragma unroll
-                for (int i = 0; i < VEC; ++i) u[i] = fmaf(wi, v[i], u[i]);
+                for (int i = 0; i < VEC; ++i) v[i] = old[o][i];
             }
-        } else {
-#pragma unroll(NS ? N : 1)
-            for (int s = 0; s < N; ++s) {
-                if (s >= n) break;
-                const float wi = in_s[s];
+            const float wi = in_s[o];
 #pragma unroll
-                for (int i = 0; i < VEC; ++i) u[i] = fmaf(wi, old[s][i], u[i]);
-            }
+            for (int i = 0; i < VEC; ++i) u[i] = fmaf(wi, v[i], u[i]);
         }
-        hc_store<VEC>(u_s + c, u);
-#pragma unroll
-        for (int i = 0; i < VEC; ++i) ss = fmaf(u[i], u[i], ss);
-    }
-    ss = ap_block_sum(ss, scratch);
-    const float inv = 1.0f / sqrtf(ss / (float)H + A.eps);
-    // a thread reads back the columns it wrote itself
-    for (int c = threadIdx.x * VEC; c < H; c += blockDim.x * VEC) {
-        float u[VEC], ww[VEC];
-        hc_load<VEC>(u_s + c, u);
+    };
+    auto store = [&](int c, float (&u)[VEC], float inv) {
+        float ww[VEC];
         hc_load<VEC>(A.w + c, ww);
 #pragma unroll
         for (int i = 0; i < VEC; ++i) u[i] = u[i] * inv * ww[i];
         hc_store<VEC>(out + (size_t)blockIdx.x * H + c, u);
+    };
+
+    float ss = 0.f;
+    if constexpr (ONE) {
+        const int c = threadIdx.x * VEC;
+        const bool in = c < H;
+        float old[N][VEC], d[HC_MAX_SLICES][VEC], y[VEC], u[VEC];
+        if (in) {
+#pragma unroll
+            for (int s = 0; s < HC_MAX_SLICES; ++s)
+                if (s < A.S) load_slice(s, c, d[s]);
+            load_old(c, old);
+        }
+        if (normed) {
+#pragma unroll
+            for (int s = 0; s < HC_MAX_SLICES; ++s)
+                if (in && s < A.S) square(s, d[s]);
+            finish_factors();
+        } else {
+            __syncthreads();                                 // the weights are in shared memory
+        }
+        if (in) {
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) y[i] = 0.f;
+#pragma unroll
+            for (int s = 0; s < HC_MAX_SLICES; ++s)
+                if (s < A.S) add_slice(s, c, d[s], y);
+            apply(c, old, y, u);
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) ss = fmaf(u[i], u[i], ss);
+        }
+        ss = ap_block_sum(ss, scratch);
+        if (in) store(c, u, 1.0f / sqrtf(ss / (float)H + A.eps));
+    } else {
+        if (normed) {
+            for (int c = threadIdx.x * VEC; c < H; c += blockDim.x * VEC) {
+#pragma unroll
+                for (int s = 0; s < HC_MAX_SLICES; ++s)
+                    if (s < A.S) {
+                        float d[VEC];
+                        load_slice(s, c, d);
+                        square(s, d);
+                    }
+            }
+            finish_factors();
+        } else {
+            __syncthreads();
+        }
+        for (int c = threadIdx.x * VEC; c < H; c += blockDim.x * VEC) {
+            float old[N][VEC], y[VEC], u[VEC];
+            load_old(c, old);
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) y[i] = 0.f;
+#pragma unroll
+            for (int s = 0; s < HC_MAX_SLICES; ++s)
+                if (s < A.S) {
+                    float d[VEC];
+                    load_slice(s, c, d);
+                    add_slice(s, c, d, y);
+                }
+            apply(c, old, y, u);
+            hc_store<VEC>(u_s + c, u);
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) ss = fmaf(u[i], u[i], ss);
+        }
+        ss = ap_block_sum(ss, scratch);
+        const float inv = 1.0f / sqrtf(ss / (float)H + A.eps);
+        // a thread reads back the columns it wrote itself
+        for (int c = threadIdx.x * VEC; c < H; c += blockDim.x * VEC) {
+            float u[VEC];
+            hc_load<VEC>(u_s + c, u);
+            store(c, u, inv);
+        }
     }
 }
 
@@ -195,25 +268,27 @@ AP_EXPORT int ap_stream_norm(float* x, const int* rows, int R, const float* delt
                      ((((uintptr_t)x) | ((uintptr_t)delta) | ((uintptr_t)slice_bias) | ((uintptr_t)slice_w) | ((uintptr_t)w)) & 15) == 0 &&
                      (((uintptr_t)out) & (out_dtype == AP_F32 ? 15 : 7)) == 0;
     int threads = ((vec ? H / 4 : H) + 31) / 32 * 32;
-    if (threads > 512) threads = 512;
-    const size_t smem = (size_t)H * sizeof(float);
+    const bool built = streams <= 4 || streams == 6 || streams == 8;       // (else the kernel for any number)
+    const bool one = built && vec && threads <= (streams <= 4 ? 1024 : 512);   // a row in one pass, kept in registers
+    if (!one && threads > 512) threads = 512;
+    const size_t smem = one ? 0 : (size_t)H * sizeof(float);
     AP_REQUIRE(smem <= 200 * 1024, "stream_norm: a row of %d does not fit shared memory", H);
     StreamNormArgs A;
     A.x = x; A.rows = rows; A.delta = delta; A.S = delta ? S : 0; A.slice_stride = (size_t)slice_stride;
     A.slice_bias = slice_bias; A.slice_w = slice_w; A.slice_eps = slice_eps; A.slice_scale = slice_scale;
     A.out_w = out_w; A.mix = mix; A.in_w = in_w; A.w = w; A.eps = eps; A.update = (update && delta) ? 1 : 0;
     A.streams = streams; A.H = H;
-#define LAUNCH(N, V, TO)                                                                                            \
+#define LAUNCH(N, V, ONE, TO)                                                                                       \
     do {                                                                                                            \
-        auto kern = stream_norm_kernel<N, V, TO>;                                                                   \
+        auto kern = stream_norm_kernel<N, V, ONE, TO>;                                                                  \
         if (smem > 40 * 1024) {                                                                                     \
             cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
             AP_REQUIRE(e == cudaSuccess, "stream_norm: cannot reserve %zu bytes of shared memory", smem);           \
         }                                                                                                           \
         AP_CHECK_PDL_LAUNCH("stream_norm", ap_launch_pdl(kern, dim3((unsigned)R), dim3(threads), smem, stream, A, (TO*)out)); \
     } while (0)
-#define LAUNCH_T(N, V) do { if (out_dtype == AP_F32) LAUNCH(N, V, float); else LAUNCH(N, V, bf16); } while (0)
-#define LAUNCH_V(N) do { if (vec) LAUNCH_T(N, 4); else LAUNCH_T(N, 1); } while (0)
+#define LAUNCH_T(N, V, ONE) do { if (out_dtype == AP_F32) LAUNCH(N, V, ONE, float); else LAUNCH(N, V, ONE, bf16); } while (0)
+#define LAUNCH_V(N) do { if (one) LAUNCH_T(N, 4, true); else if (vec) LAUNCH_T(N, 4, false); else LAUNCH_T(N, 1, false); } while (0)
     AP_REQUIRE(out_dtype == AP_F32 || out_dtype == AP_BF16, "stream_norm: unknown dtype %d", out_dtype);
     switch (streams) {
         case 1: LAUNCH_V(1); break;
@@ -222,7 +297,7 @@ AP_EXPORT int ap_stream_norm(float* x, const int* rows, int R, const float* delt
         case 4: LAUNCH_V(4); break;
         case 6: LAUNCH_V(6); break;
         case 8: LAUNCH_V(8); break;
-        default: LAUNCH_T(0, 1);
+        default: LAUNCH_T(0, 1, false);
     }
 #undef LAUNCH_V
 #undef LAUNCH_T

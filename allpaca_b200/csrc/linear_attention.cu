@@ -19,6 +19,9 @@
 // coordinate or none), times silu(gate) or sigmoid(gate), times a constant, rounded to the activation type for the
 // output projection.
 //
+// A step of single rows (decoding) runs the recurrence as written (la_scan_kernel); a step of portions runs it eight
+// tokens at a time (la_blocks_kernel, la_chunk_kernel).
+//
 // Everything is 32-bit: inputs are 32-bit sums of the projections, decays, exponentials, the state, the
 // read-out and the norm.  A sequence's rows are found through seq_start, its state row through
 // state_slots; a portion whose first row has position 0 starts from zeros.  Nothing is decided on the
@@ -295,6 +298,566 @@ __global__ void __launch_bounds__(128) la_scan_kernel(const LaScanArgs A) {
     }
 }
 
+// ---- the recurrence, eight tokens at a time -------------------------------------------------
+// What a prompt's portion takes instead of the chain above.  Over a block of tokens the recurrence closes into sums that
+// need the state only as it was before them.  With c_r the decays of token r (a vector over the key channels, or a number),
+// C_r = c_0 .. c_r their running product and c(j, r) = c_{j+1} .. c_r what is left of token j's write at token r:
+//
+//   u_r = beta_r (v_r - S^T (C_r k_r) - sum_{j<r} [k_r . c(j, r) k_j] u_j)          (delta rule; else u_r = v_r)
+//   o_r = S^T (C_r q_r) + sum_{j<=r} [q_r . c(j, r) k_j] u_j
+//   S  <- C_7 S + sum_j (c(j, 7) k_j) u_j^T
+//
+// The bracketed numbers and the vectors with their decays do not depend on the state: la_blocks_kernel forms them once
+// per (eight tokens, head), together with everything the rows need before the recurrence (rotation, unit vectors, SiLU,
+// decays, gates), and leaves them in one block of scratch.  The recurrence's chain is then one step per EIGHT tokens, whose
+// sums meet over the lanes in the same rounds of shuffles, and a state entry costs three multiply-adds a token, two entries
+// to an instruction.  All 32-bit, products of decays included (none is ever divided by).  A block of fewer tokens is filled
+// up with tokens that do nothing.
+//
+// A block: the numbers (REC_*), then rows C_r k_r, rows C_r q_r, for decays per channel also rows c(j, 7) k_j and the row
+// C_7, each padded with zeros to DS = PER * NP numbers, then rows of values (times beta) padded to VS.  The block of
+// (sequence s, rows 8i .. of its portion, head h) lies at index (seq_start[s] / 8 + i + s) * heads + h.
+#define LT 8                     // tokens of a block
+#define REC_BA 0                 // beta_r * C_r (C_r is 1 here where the vectors hold it)
+#define REC_A (REC_BA + LT)      // rows r = 1 .. 7: beta_r [k_r . c(j, r) k_j], j < r, in runs of four
+#define REC_GAMMA (REC_A + 40)   // c(r, 7)
+#define REC_ALPHA (REC_GAMMA + LT)   // C_r * out_scale
+#define REC_P (REC_ALPHA + LT)   // rows r = 0 .. 7: [q_r . c(j, r) k_j] * out_scale, zero for j > r
+#define REC_TOTAL (REC_P + LT * LT)  // C_7
+#define REC_SIZE (REC_TOTAL + 4)
+#define PAIRS_BELOW (LT * (LT - 1) / 2)
+__host__ __device__ constexpr int rec_a_row(int r) { return REC_A + (r <= 4 ? (r - 1) * 4 : 16 + (r - 5) * 8); }
+
+#define LC_WARPS_WANTED 400L     // warps a step of portions should bring to the GPU's schedulers
+
+struct LaBlocks { float* at; int DS, VS, size; };
+
+// (first row, rows, place in the scratch) of the b-th block; false beyond the last
+__device__ __forceinline__ bool lc_find(const int* seq_start, int nseq, int b, int& row, int& cnt, int& index) {
+    for (int s = 0; s < nseq; ++s) {
+        const int a = seq_start[s], n = seq_start[s + 1] - a, groups = (n + LT - 1) / LT;
+        if (b < groups) {
+            row = a + b * LT;
+            cnt = min(LT, n - b * LT);
+            index = a / LT + b + s;
+            return true;
+        }
+        b -= groups;
+    }
+    return false;
+}
+
+// Sums over a warp's lanes of N numbers (a multiple of 32): every round halves what a lane holds; lane l ends with
+// the sums of numbers l * N / 32 .. in places 0 ..
+template <int N> __device__ __forceinline__ void la_scatter_sums(float (&v)[N], int lane) {
+#pragma unroll
+    for (int n = N / 2, o = 16; o >= 1; n >>= 1, o >>= 1) {
+        const bool up = (lane & o) != 0;
+#pragma unroll
+        for (int i = 0; i < N / 2; ++i) {
+            if (i < n) {
+                const float send = up ? v[i] : v[i + n], keep = up ? v[i + n] : v[i];
+                v[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+            }
+        }
+    }
+}
+
+// One CTA per (block of tokens, head), a channel to a thread.  CH: 0, DECAY_CHANNEL or DECAY_CHANNEL_TOKEN.
+template <int CH>
+__global__ void __launch_bounds__(128, 4) la_blocks_kernel(const LaScanArgs A, const LaBlocks B, int nseq) {
+    __shared__ float red[4][2 * 32], numbers[2][LT], unit_s[2 * LT];
+    ap_pdl_wait();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
+    const int H = A.heads, D = A.D, V = A.V, DS = B.DS, VS = B.VS;
+    const int h = (int)(blockIdx.x % H), g = h / (H / A.qk_heads);
+    int row, cnt, index;
+    if (!lc_find(A.seq_start, nseq, (int)(blockIdx.x / H), row, cnt, index)) return;
+    float* rec = B.at + ((size_t)index * H + h) * B.size;
+    float* kt = rec + REC_SIZE;
+    float* qt = kt + LT * DS;
+    float* kh = qt + LT * DS;
+    float* ct = kh + LT * DS;
+    float* vb = CH ? ct + DS : kh;
+    const bool delta = A.beta != nullptr;
+    const int mode = A.qk_mode, half = A.rot_dims / 2;
+    const float* qp = A.q + (size_t)row * A.ld_q + (size_t)g * D;
+    const float* kp = A.k + (size_t)row * A.ld_k + (size_t)g * D;
+    const float* zp = CH ? A.decay_channel + (size_t)row * A.ld_dc + (size_t)h * D : nullptr;
+    // the numbers of each token: gate of the write, decay of the head (1 where channels have their own)
+    if (threadIdx.x < LT) {
+        const int r = threadIdx.x;
+        const size_t t = (size_t)row + r;
+        float b = r < cnt ? 1.f : 0.f, a = 1.f;
+        if (r < cnt) {
+            if (delta) b = 1.0f / (1.0f + expf(-A.beta[t * A.ld_beta + h]));
+            if (A.decay_mode == DECAY_HEAD_CONST) a = A.decay_const[h];
+            if (A.decay_mode == DECAY_HEAD_TOKEN)
+                a = expf(-expf(A.decay_const[h]) * la_softplus(A.decay_head[t * A.ld_dh + h] + (A.dt_bias ? A.dt_bias[h] : 0.f)));
+        }
+        numbers[0][r] = b;
+        numbers[1][r] = a;
+    }
+    if (mode == QK_UNIT) {
+        float ss[32];
+#pragma unroll
+        for (int i = 0; i < 32; ++i) ss[i] = 0.f;
+        for (int d = threadIdx.x; d < D; d += blockDim.x) {
+#pragma unroll
+            for (int r = 0; r < LT; ++r) {
+                const float q = r < cnt ? qp[r * A.ld_q + d] : 0.f, k = r < cnt ? kp[r * A.ld_k + d] : 0.f;
+                ss[r] = fmaf(q, q, ss[r]);
+                ss[LT + r] = fmaf(k, k, ss[LT + r]);
+            }
+        }
+        la_scatter_sums<32>(ss, lane);
+        if (lane < 2 * LT) red[warp][lane] = ss[0];
+        __syncthreads();
+        if (threadIdx.x < 2 * LT) {
+            float sum = 0.f;
+            for (int w = 0; w < nwarps; ++w) sum += red[w][threadIdx.x];
+            unit_s[threadIdx.x] = 1.0f / sqrtf(sum + A.unit_eps);
+        }
+    }
+    __syncthreads();
+    const float rate = CH == DECAY_CHANNEL_TOKEN ? expf(A.decay_const[h]) : 0.f;
+    float acc[64];                                           // pairs j < r of keys, then pairs j <= r of queries and keys
+#pragma unroll
+    for (int i = 0; i < 64; ++i) acc[i] = 0.f;
+    for (int d = threadIdx.x; d < DS; d += blockDim.x) {
+        float q[LT], k[LT], c[LT];
+#pragma unroll
+        for (int r = 0; r < LT; ++r) {
+            const bool in = r < cnt && d < D;
+            q[r] = in ? qp[r * A.ld_q + d] : 0.f;
+            k[r] = in ? kp[r * A.ld_k + d] : 0.f;
+            c[r] = (CH && in) ? zp[r * A.ld_dc + d] : 0.f;
+        }
+        if (mode == QK_UNIT) {
+#pragma unroll
+            for (int r = 0; r < LT; ++r) { q[r] *= unit_s[r]; k[r] *= unit_s[LT + r]; }
+        } else if (mode == QKV_SILU) {
+#pragma unroll
+            for (int r = 0; r < LT; ++r) { q[r] = la_silu(q[r]); k[r] = la_silu(k[r]); }
+        } else if (mode == QK_ROTATE && d < A.rot_dims) {
+            const int m = d < half ? d : d - half, partner = d < half ? d + half : d - half;
+#pragma unroll
+            for (int r = 0; r < LT; ++r) {
+                if (r < cnt) {
+                    const float2 cs = *reinterpret_cast<const float2*>(A.cos_sin + (((size_t)row + r) * half + m) * 2);
+                    const float sn = d < half ? -cs.y : cs.y;
+                    q[r] = q[r] * cs.x + qp[r * A.ld_q + partner] * sn;
+                    k[r] = k[r] * cs.x + kp[r * A.ld_k + partner] * sn;
+                }
+            }
+        }
+        if (CH) {
+            const float bias = (CH == DECAY_CHANNEL_TOKEN && A.dt_bias && d < D) ? A.dt_bias[(size_t)h * D + d] : 0.f;
+#pragma unroll
+            for (int r = 0; r < LT; ++r) {
+                const float e = CH == DECAY_CHANNEL ? expf(-la_softplus(-c[r]) * A.inv_tau) : expf(-rate * la_softplus(c[r] + bias));
+                c[r] = r < cnt ? e : 1.f;
+            }
+        }
+        // kk[j] becomes c(j, r) k_j as r goes on
+        float kk[LT], upto = 1.f;
+        int below = 0, upon = PAIRS_BELOW;
+#pragma unroll
+        for (int r = 0; r < LT; ++r) {
+            if (CH) {
+                upto *= c[r];
+#pragma unroll
+                for (int j = 0; j < r; ++j) kk[j] *= c[r];
+            }
+            kk[r] = k[r];
+#pragma unroll
+            for (int j = 0; j < r; ++j) {
+                acc[below + j] = fmaf(k[r], kk[j], acc[below + j]);
+                acc[upon + j] = fmaf(q[r], kk[j], acc[upon + j]);
+            }
+            acc[upon + r] = fmaf(q[r], k[r], acc[upon + r]);
+            below += r;
+            upon += r + 1;
+            kt[r * DS + d] = CH ? upto * k[r] : k[r];
+            qt[r * DS + d] = CH ? upto * q[r] : q[r];
+        }
+        if (CH) {
+#pragma unroll
+            for (int r = 0; r < LT; ++r) kh[r * DS + d] = kk[r];
+            ct[d] = d < D ? upto : 0.f;
+        }
+    }
+    la_scatter_sums<64>(acc, lane);
+    red[warp][2 * lane] = acc[0];
+    red[warp][2 * lane + 1] = acc[1];
+    __syncthreads();
+    const float* beta = numbers[0];
+    const float* a = numbers[1];
+    for (int t = threadIdx.x; t < LT * LT; t += blockDim.x) {
+        float sum = 0.f;
+        for (int w = 0; w < nwarps; ++w) sum += red[w][t];
+        // number t is (r, j): t = r (r - 1) / 2 + j below the diagonal, then r (r + 1) / 2 + j with it
+        const bool keys = t < PAIRS_BELOW;
+        int r = keys ? 1 : 0, j = keys ? t : t - PAIRS_BELOW;
+        while (j >= (keys ? r : r + 1)) { j -= keys ? r : r + 1; ++r; }
+        float left = 1.f;                                    // what the head's decays leave of token j at token r
+        for (int i = j + 1; i <= r; ++i) left *= a[i];
+        if (keys) rec[(r <= 4 ? REC_A + (r - 1) * 4 : REC_A + 16 + (r - 5) * 8) + j] = beta[r] * left * sum;
+        else rec[REC_P + r * LT + j] = A.out_scale * left * sum;
+        if ((t & (LT - 1)) > t / LT) rec[REC_P + t] = 0.f;   // a later token's write
+    }
+    if (threadIdx.x < LT) {
+        const int r = threadIdx.x;
+        float upto = 1.f, after = 1.f;
+        for (int i = 0; i < LT; ++i) {
+            if (i <= r) upto *= a[i];
+            else after *= a[i];
+        }
+        rec[REC_BA + r] = beta[r] * upto;
+        rec[REC_GAMMA + r] = after;
+        rec[REC_ALPHA + r] = upto * A.out_scale;
+        if (r == LT - 1) rec[REC_TOTAL] = upto;
+    }
+    for (int r = 0; r < LT; ++r) {
+        const float* vp = A.v + ((size_t)row + r) * A.ld_v + (size_t)h * V;
+        for (int d = threadIdx.x; d < VS; d += blockDim.x) {
+            float v = (r < cnt && d < V) ? vp[d] : 0.f;
+            if (mode == QKV_SILU) v = la_silu(v);
+            vb[r * VS + d] = delta ? beta[r] * v : v;
+        }
+    }
+}
+
+// two 32-bit numbers to a register pair, multiplied and added in one instruction
+typedef unsigned long long la_pair;
+__device__ __forceinline__ la_pair la_fma2(la_pair a, la_pair b, la_pair c) {
+    la_pair d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ la_pair la_mul2(la_pair a, la_pair b) {
+    la_pair d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ la_pair la_pack(float lo, float hi) {
+    la_pair d;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+    return d;
+}
+__device__ __forceinline__ float2 la_unpack(la_pair p) {
+    float2 v;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(v.x), "=f"(v.y) : "l"(p));
+    return v;
+}
+__device__ __forceinline__ float la_sum2(la_pair p) { const float2 v = la_unpack(p); return v.x + v.y; }
+
+// One CTA per (sequence, head, block of value columns).  NP lanes share CPT columns; a lane holds PER entries of each
+// (entry i of lane p is row (i / 4) * 4 NP + 4 p + i % 4), so that a vector read from shared memory serves CPT columns: what
+// bounds this kernel is the width of shared memory, one 128-byte wavefront per number and warp, and repeated addresses
+// within a warp do not make a 16-byte read cheaper.  A lane keeps its columns in an order of its own, column c ^ (p mod
+// CPT) in place c: in the first rounds of the sums over the lanes a lane then always sends the upper half of what it holds
+// and keeps the lower, without choosing, and ends with the numbers of column p mod CPT, whose writes u it works out
+// together with the M = NP / CPT lanes that ended on the same column.  `stage` blocks of eight tokens at a time come
+// through two shared-memory buffers.
+template <int PER, int NP, int CPT, bool CHANNEL, bool DELTA>
+__global__ void __launch_bounds__(128, 1) la_chunk_kernel(const LaScanArgs A, const LaBlocks B, int stage) {
+    extern __shared__ __align__(16) float sm[];
+    ap_pdl_wait();
+    const int s = blockIdx.x, h = blockIdx.y;
+    const int a = A.seq_start[s], n = A.seq_start[s + 1] - a;
+    if (n <= 0) return;
+    constexpr int DS = PER * NP, MAIN = REC_SIZE + (CHANNEL ? 3 * LT + 1 : 2 * LT) * DS;
+    constexpr int COLS = 128 / NP * CPT, M = NP / CPT, ONE = MAIN + LT * COLS;
+    const int D = A.D, V = A.V, VS = B.VS;
+    const int col0 = blockIdx.z * COLS;
+    const int vcols = min(COLS, VS - col0);                   // columns to bring: whole 16-byte runs
+    const int part = threadIdx.x % NP, swap = part % CPT, idx = part / CPT;
+    const int first = threadIdx.x / NP * CPT;                 // this lane's columns in the block: first + (c ^ swap)
+    float* st = A.state + (size_t)A.state_slots[s] * A.state_stride + (size_t)h * D * V + col0 + first;
+    const bool fresh = A.positions[a] == 0;
+    la_pair S[CPT][PER / 2];
+#pragma unroll
+    for (int c = 0; c < CPT; ++c) {
+        const bool live = col0 + first + (c ^ swap) < V;
+#pragma unroll
+        for (int i = 0; i < PER / 2; ++i) {
+            float e[2];
+#pragma unroll
+            for (int k = 0; k < 2; ++k) {
+                const int m = 2 * i + k, nn = (m >> 2) * 4 * NP + 4 * part + (m & 3);
+                e[k] = (!fresh && live && nn < D) ? st[(size_t)nn * V + (c ^ swap)] : 0.f;
+            }
+            S[c][i] = la_pack(e[0], e[1]);
+        }
+    }
+    const int groups = (n + LT - 1) / LT;
+    const float* src = B.at + ((size_t)(a / LT + s) * A.heads + h) * B.size;
+    const size_t step = (size_t)A.heads * B.size;
+
+    auto fetch = [&](int g0, float* buf) {
+        const int cnt = min(stage, groups - g0);
+        for (int g = 0; g < cnt; ++g) {
+            const float* from = src + (size_t)(g0 + g) * step;
+            float* to = buf + g * ONE;
+#pragma unroll
+            for (int i = 0; i < (MAIN + 511) / 512; ++i) {
+                const int at = (i * 128 + threadIdx.x) * 4;
+                if (at < MAIN) la_copy16(to + at, from + at);
+            }
+            const float* vfrom = from + MAIN + col0;
+            for (int i = threadIdx.x; i < LT * (COLS / 4); i += 128) {
+                const int r = i / (COLS / 4), c = i % (COLS / 4) * 4;
+                if (c < vcols) la_copy16(to + MAIN + r * COLS + c, vfrom + (size_t)r * VS + c);
+            }
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+
+    // the token (or the tokens, with fewer lanes to a column) whose read-out of this lane's column it finishes; of the
+    // lanes that end with the same one the first stores it
+    constexpr int QN = M >= LT ? 1 : LT / M;
+    int q_first = 0;
+#pragma unroll
+    for (int o = M >> 1, n2 = LT >> 1; o > 0 && n2 > 0; o >>= 1, n2 >>= 1) q_first += (idx & o) ? n2 : 0;
+    const bool writer = col0 + first + swap < V && (M <= LT || (idx & (M / LT - 1)) == 0);
+    float* yp = A.y + (size_t)a * A.ld_y + (size_t)h * V + col0 + first + swap;
+
+    fetch(0, sm);
+    int which = 0;
+    for (int g0 = 0; g0 < groups; g0 += stage, which ^= 1) {
+        const int cnt = min(stage, groups - g0);
+        float* buf = sm + which * stage * ONE;
+        if (g0 + stage < groups) {
+            fetch(g0 + stage, sm + (which ^ 1) * stage * ONE);
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+        } else {
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+        }
+        __syncthreads();
+        for (int g = 0; g < cnt; ++g) {
+            const float* rec = buf + g * ONE;
+            const float* kt = rec + REC_SIZE + 4 * part;
+            const float* qt = kt + LT * DS;
+            const float* kh = CHANNEL ? qt + LT * DS : kt;
+            const float* ct = kh + LT * DS;
+            const float* vs = rec + MAIN + first + swap;
+            float kd[LT][CPT], qd[LT][CPT];
+#pragma unroll
+            for (int r = 0; r < LT; ++r) {
+                la_pair ak[CPT], aq[CPT];
+#pragma unroll
+                for (int i = 0; i < PER / 4; ++i) {
+                    const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(qt + r * DS + i * 4 * NP);
+#pragma unroll
+                    for (int c = 0; c < CPT; ++c) {
+                        aq[c] = i == 0 ? la_mul2(S[c][0], q.x) : la_fma2(S[c][2 * i], q.x, aq[c]);
+                        aq[c] = la_fma2(S[c][2 * i + 1], q.y, aq[c]);
+                    }
+                    if (DELTA) {
+                        const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(kt + r * DS + i * 4 * NP);
+#pragma unroll
+                        for (int c = 0; c < CPT; ++c) {
+                            ak[c] = i == 0 ? la_mul2(S[c][0], k.x) : la_fma2(S[c][2 * i], k.x, ak[c]);
+                            ak[c] = la_fma2(S[c][2 * i + 1], k.y, ak[c]);
+                        }
+                    }
+                }
+#pragma unroll
+                for (int c = 0; c < CPT; ++c) {
+                    qd[r][c] = la_sum2(aq[c]);
+                    kd[r][c] = DELTA ? la_sum2(ak[c]) : 0.f;
+                }
+            }
+            // the sums over the lanes: first the columns part ways ...
+#pragma unroll
+            for (int o = CPT >> 1; o > 0; o >>= 1)
+#pragma unroll
+                for (int r = 0; r < LT; ++r)
+#pragma unroll
+                    for (int c = 0; c < o; ++c) {
+                        if (DELTA) kd[r][c] += __shfl_xor_sync(0xffffffffu, kd[r][c + o], o);
+                        qd[r][c] += __shfl_xor_sync(0xffffffffu, qd[r][c + o], o);
+                    }
+            // ... then the keys' sums end on every lane of a column, the queries' on one lane (or a few) to a token
+            if (DELTA) {
+#pragma unroll
+                for (int o = M >> 1; o > 0; o >>= 1)
+#pragma unroll
+                    for (int r = 0; r < LT; ++r) kd[r][0] += __shfl_xor_sync(0xffffffffu, kd[r][0], o * CPT);
+            }
+            float qs[LT], u[LT];
+#pragma unroll
+            for (int r = 0; r < LT; ++r) { qs[r] = qd[r][0]; u[r] = vs[r * COLS]; }
+#pragma unroll
+            for (int o = M >> 1, n2 = LT >> 1; o > 0; o >>= 1, n2 >>= 1) {
+                if (n2 > 0) {
+                    const bool up = (idx & o) != 0;
+#pragma unroll
+                    for (int i = 0; i < LT / 2; ++i) {
+                        if (i < n2) {
+                            const float send = up ? qs[i] : qs[i + n2], keep = up ? qs[i + n2] : qs[i];
+                            qs[i] = keep + __shfl_xor_sync(0xffffffffu, send, o * CPT);
+                        }
+                    }
+                } else {
+                    qs[0] += __shfl_xor_sync(0xffffffffu, qs[0], o * CPT);
+                }
+            }
+            if (DELTA) {
+                float num[REC_GAMMA];                        // beta C and the rows of earlier tokens' shares, 16 bytes a read
+#pragma unroll
+                for (int i = 0; i < REC_GAMMA; i += 4)
+                    *reinterpret_cast<float4*>(num + i) = *reinterpret_cast<const float4*>(rec + i);
+#pragma unroll
+                for (int r = 0; r < LT; ++r) u[r] = fmaf(-num[REC_BA + r], kd[r][0], u[r]);
+#pragma unroll
+                for (int j = 0; j + 1 < LT; ++j)
+#pragma unroll
+                    for (int r = j + 1; r < LT; ++r) u[r] = fmaf(-num[rec_a_row(r) + j], u[j], u[r]);
+            }
+            // the write of every column this lane holds (with what the head's decays leave of it, where the vectors
+            // hold none)
+            float w[LT];
+            if (CHANNEL) {
+#pragma unroll
+                for (int r = 0; r < LT; ++r) w[r] = u[r];
+            } else {
+#pragma unroll
+                for (int r = 0; r < LT; ++r) w[r] = rec[REC_GAMMA + r] * u[r];
+            }
+            la_pair w2[LT][CPT];
+#pragma unroll
+            for (int r = 0; r < LT; ++r)
+#pragma unroll
+                for (int c = 0; c < CPT; ++c) {
+                    const float x = c == 0 ? w[r] : __shfl_xor_sync(0xffffffffu, w[r], c);
+                    w2[r][c] = la_pack(x, x);
+                }
+            const float total = rec[REC_TOTAL];
+            const la_pair tot2 = la_pack(total, total);
+#pragma unroll
+            for (int i = 0; i < PER / 4; ++i) {
+                ulonglong2 d = make_ulonglong2(tot2, tot2);
+                if (CHANNEL) d = *reinterpret_cast<const ulonglong2*>(ct + i * 4 * NP);
+#pragma unroll
+                for (int c = 0; c < CPT; ++c) {
+                    S[c][2 * i] = la_mul2(S[c][2 * i], d.x);
+                    S[c][2 * i + 1] = la_mul2(S[c][2 * i + 1], d.y);
+                }
+#pragma unroll
+                for (int r = 0; r < LT; ++r) {
+                    const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(kh + r * DS + i * 4 * NP);
+#pragma unroll
+                    for (int c = 0; c < CPT; ++c) {
+                        S[c][2 * i] = la_fma2(k.x, w2[r][c], S[c][2 * i]);
+                        S[c][2 * i + 1] = la_fma2(k.y, w2[r][c], S[c][2 * i + 1]);
+                    }
+                }
+            }
+            const int t0 = (g0 + g) * LT;
+#pragma unroll
+            for (int i = 0; i < QN; ++i) {
+                const int r = q_first + i;
+                float y = rec[REC_ALPHA + r] * qs[i];
+#pragma unroll
+                for (int j = 0; j < LT; j += 4) {
+                    const float4 p = *reinterpret_cast<const float4*>(rec + REC_P + LT * r + j);
+                    y = fmaf(p.w, u[j + 3], fmaf(p.z, u[j + 2], fmaf(p.y, u[j + 1], fmaf(p.x, u[j], y))));
+                }
+                if (writer && t0 + r < n) yp[(size_t)(t0 + r) * A.ld_y] = y;
+            }
+        }
+        __syncthreads();                                     // this buffer is filled again two stages on
+    }
+#pragma unroll
+    for (int c = 0; c < CPT; ++c) {
+        if (col0 + first + (c ^ swap) >= V) continue;
+#pragma unroll
+        for (int i = 0; i < PER / 2; ++i) {
+            const float2 e = la_unpack(S[c][i]);
+#pragma unroll
+            for (int k = 0; k < 2; ++k) {
+                const int m = 2 * i + k, nn = (m >> 2) * 4 * NP + 4 * part + (m & 3);
+                if (nn < D) st[(size_t)nn * V + (c ^ swap)] = k ? e.y : e.x;
+            }
+        }
+    }
+}
+
+// State entries to threads: as few lanes to a column as hold it (up to 16 entries a thread: the fewest instructions
+// per state entry); more of them (shorter chains per thread, more warps) only while the step's columns leave
+// schedulers without a warp.
+static void la_plan(int nseq, int heads, int D, int V, int& NP, int& per) {
+    NP = 1;
+    while (NP * LA_PER_MAX < D) NP *= 2;
+    while (NP < 32 && NP * 4 < D && (long long)nseq * heads * V * NP / 32 < 148 * 4) NP *= 2;
+    per = ((D + NP - 1) / NP + 3) / 4 * 4;
+    per = per <= 4 ? 4 : (per <= 8 ? 8 : LA_PER_MAX);
+}
+// whether a step of T rows goes eight tokens at a time: where its sequences bring several rows
+static bool la_in_blocks(int T, int nseq) { return T > 2 * nseq; }
+
+// The same for la_chunk_kernel: keys over as many lanes as give each four entries of a column (up to 32 lanes), and as
+// many columns to a lane as still leave every scheduler a warp.
+static void lc_plan(int nseq, int heads, int D, int V, int& NP, int& per, int& cpt) {
+    NP = 1;
+    while (NP < 32 && NP * 4 < D) NP *= 2;
+    per = D <= NP * 4 ? 4 : (D <= NP * 8 ? 8 : LA_PER_MAX);
+    cpt = NP < 4 ? 1 : ((long long)nseq * heads * V * NP / 32 >= LC_WARPS_WANTED * 4 ? 4 : 2);
+}
+
+// numbers of scratch per (block of eight tokens, head) that ap_linear_scan takes for such a step; 0: it takes none
+AP_EXPORT int ap_linear_scan_block(int T, int nseq, int heads, int D, int V, int decay_mode) {
+    if (T <= 0 || nseq <= 0 || heads <= 0 || D <= 0 || V <= 0 || !la_in_blocks(T, nseq)) return 0;
+    int NP, per, cpt;
+    lc_plan(nseq, heads, D, V, NP, per, cpt);
+    return REC_SIZE + (decay_mode >= DECAY_CHANNEL ? 3 * LT + 1 : 2 * LT) * per * NP + LT * ((V + 3) / 4 * 4);
+}
+
+typedef void (*la_chunk_fn)(const LaScanArgs, const LaBlocks, int);
+template <bool CHANNEL, bool DELTA> static la_chunk_fn lc_pick(int per, int NP, int cpt) {
+#define LC_PICK(P, N) if (per == P && NP == N) return cpt == 4 ? la_chunk_kernel<P, N, 4, CHANNEL, DELTA> : la_chunk_kernel<P, N, 2, CHANNEL, DELTA>
+    LC_PICK(4, 4); LC_PICK(4, 8); LC_PICK(4, 16); LC_PICK(4, 32); LC_PICK(8, 32); LC_PICK(LA_PER_MAX, 32);
+#undef LC_PICK
+    return NP == 1 ? la_chunk_kernel<4, 1, 1, CHANNEL, DELTA> : la_chunk_kernel<4, 2, 1, CHANNEL, DELTA>;
+}
+
+static int la_run_blocks(LaScanArgs& A, int nseq, float* scratch, cudaStream_t stream) {
+    int NP, per, cpt;
+    lc_plan(nseq, A.heads, A.D, A.V, NP, per, cpt);
+    LaBlocks B;
+    B.at = scratch;
+    B.DS = per * NP;
+    B.VS = (A.V + 3) / 4 * 4;
+    const bool channel = A.decay_mode >= DECAY_CHANNEL, delta = A.beta != nullptr;
+    const int main_floats = REC_SIZE + (channel ? 3 * LT + 1 : 2 * LT) * B.DS;
+    B.size = main_floats + LT * B.VS;
+    const int cols = 128 / NP * cpt;
+    const dim3 grid((unsigned)nseq, (unsigned)A.heads, (unsigned)((A.V + cols - 1) / cols));
+    int stage = 2;
+    size_t smem;
+    while ((smem = 2 * (size_t)stage * (main_floats + LT * cols) * sizeof(float)) > 100 * 1024 && stage > 1) stage /= 2;
+    AP_REQUIRE(smem <= 200 * 1024 && grid.z <= 65535, "linear_scan: keys of %d do not fit the staging buffers", A.D);
+    const long long units = ((long long)A.T / LT + nseq) * A.heads;
+    AP_REQUIRE(units <= 0x7fffffffLL, "linear_scan: %d rows of %d heads exceed the grid", A.T, A.heads);
+    int threads = (A.D + 31) / 32 * 32;
+    if (threads > 128) threads = 128;
+    auto blocks = A.decay_mode == DECAY_CHANNEL ? la_blocks_kernel<DECAY_CHANNEL>
+                : A.decay_mode == DECAY_CHANNEL_TOKEN ? la_blocks_kernel<DECAY_CHANNEL_TOKEN> : la_blocks_kernel<0>;
+    AP_CHECK_PDL_LAUNCH("linear_scan (blocks)", ap_launch_pdl(blocks, dim3((unsigned)units), dim3(threads), 0, stream, A, B, nseq));
+    la_chunk_fn kern = channel ? (delta ? lc_pick<true, true>(per, NP, cpt) : lc_pick<true, false>(per, NP, cpt))
+                               : (delta ? lc_pick<false, true>(per, NP, cpt) : lc_pick<false, false>(per, NP, cpt));
+    if (smem > 48 * 1024) {
+        cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        AP_REQUIRE(e == cudaSuccess, "linear_scan: cannot reserve %zu bytes of shared memory", smem);
+    }
+    // the kernel before does not let this one start early: CTAs placed while others still hold most SMs would crowd
+    // on the few that are free, and a chain this long does not recover from that
+    AP_CHECK_PDL_LAUNCH("linear_scan (eight tokens at a time)", ap_launch_pdl(kern, grid, dim3(128), smem, stream, A, B, stage));
+    return AP_OK;
+}
+
 AP_EXPORT int ap_linear_scan(float* q, long long ld_q, float* k, long long ld_k, float* v,
                              long long ld_v, float* decay_channel, long long ld_dc, float* decay_head,
                              long long ld_dh, const float* decay_const, const float* dt_bias, float* beta,
@@ -302,7 +865,7 @@ AP_EXPORT int ap_linear_scan(float* q, long long ld_q, float* k, long long ld_k,
                              long long state_stride, const int* seq_start, const int* positions,
                              const int* state_slots, float* y, long long ld_y, int T, int nseq, int heads,
                              int qk_heads, int D, int V, int decay_mode, int qk_mode, float tau, float unit_eps,
-                             float out_scale, cudaStream_t stream) {
+                             float out_scale, float* scratch, cudaStream_t stream) {
     AP_REQUIRE(T >= 0 && nseq >= 0 && heads > 0 && qk_heads > 0 && heads % qk_heads == 0 && D > 0 && V > 0,
                "linear_scan: bad sizes heads=%d qk_heads=%d key=%d value=%d", heads, qk_heads, D, V);
     AP_REQUIRE(D <= LA_PER_MAX * 32, "linear_scan: keys of %d exceed %d", D, LA_PER_MAX * 32);
@@ -316,15 +879,10 @@ AP_EXPORT int ap_linear_scan(float* q, long long ld_q, float* k, long long ld_k,
     AP_REQUIRE(qk_mode == QK_PLAIN || qk_mode == QK_UNIT || qk_mode == QKV_SILU ||
                (qk_mode == QK_ROTATE && cos_sin && rot_dims > 0 && rot_dims % 2 == 0 && rot_dims <= D),
                "linear_scan: query/key mode %d with %d rotated coordinates of %d", qk_mode, rot_dims, D);
+    AP_REQUIRE((((uintptr_t)scratch) & 15) == 0, "linear_scan: the scratch must start on a 16-byte boundary");
     if (T == 0 || nseq == 0) return AP_OK;
-    // as few lanes to a column as hold it (up to 16 entries a thread: the fewest instructions per state entry);
-    // more of them (shorter chains per thread, more warps) only while the step's columns leave schedulers without
-    // a warp (measured: with four warps to a scheduler and four entries a thread the longer reductions cost more
-    // than the other warps hide, 733 -> 797 us for 2048 tokens of the delta rule on 16 heads of 128 x 128)
-    int NP = 1;
-    while (NP * LA_PER_MAX < D) NP *= 2;
-    while (NP < 32 && NP * 4 < D && (long long)nseq * heads * V * NP / 32 < 148 * 4) NP *= 2;
-    const int per = ((D + NP - 1) / NP + 3) / 4 * 4;
+    int NP, per;
+    la_plan(nseq, heads, D, V, NP, per);
     int cols = 128 / NP;
     if (cols > V) cols = V;
     int threads = (cols * NP + 31) / 32 * 32;
@@ -346,6 +904,7 @@ AP_EXPORT int ap_linear_scan(float* q, long long ld_q, float* k, long long ld_k,
     A.T = T; A.heads = heads; A.qk_heads = qk_heads; A.D = D; A.V = V; A.NP = NP; A.cols = cols;
     A.decay_mode = decay_mode; A.qk_mode = qk_mode; A.vec = vec;
     A.inv_tau = decay_mode == DECAY_CHANNEL ? 1.0f / tau : 0.f; A.unit_eps = unit_eps; A.out_scale = out_scale;
+    if (scratch != nullptr && la_in_blocks(T, nseq)) return la_run_blocks(A, nseq, scratch, stream);
     const int units = (qk_mode == QK_PLAIN ? 0 : 2 * qk_heads) + (qk_mode == QKV_SILU ? heads : 0) + (channel ? heads : 0) +
                       ((decay_mode == DECAY_HEAD_TOKEN || beta != nullptr) ? 1 : 0);
     if (units > 0) {
@@ -353,12 +912,11 @@ AP_EXPORT int ap_linear_scan(float* q, long long ld_q, float* k, long long ld_k,
         AP_CHECK_PDL_LAUNCH("linear_scan (rows made ready)",
                             ap_launch_pdl(la_prepare_kernel, dim3((unsigned)blocks), dim3(128), 0, stream, A));
     }
-    const int per_built = per <= 4 ? 4 : (per <= 8 ? 8 : LA_PER_MAX);
-    const size_t smem = 2 * ((size_t)LA_CHUNK * ((cols + 3) / 4 * 4 + (channel ? 3 : 2) * (per_built * NP)) + 2 * LA_CHUNK) *
+    const size_t smem = 2 * ((size_t)LA_CHUNK * ((cols + 3) / 4 * 4 + (channel ? 3 : 2) * (per * NP)) + 2 * LA_CHUNK) *
                         sizeof(float);
     void (*kern)(const LaScanArgs) = nullptr;
 #define LA_PICK(P)                                                                                     \
-    if (per_built == P)                                                                                \
+    if (per == P)                                                                                      \
         kern = NP == 1 ? la_scan_kernel<P, 1> : NP == 2 ? la_scan_kernel<P, 2> : NP == 4 ? la_scan_kernel<P, 4> \
              : NP == 8 ? la_scan_kernel<P, 8> : NP == 16 ? la_scan_kernel<P, 16> : la_scan_kernel<P, 32>;
     LA_PICK(4) LA_PICK(8) LA_PICK(LA_PER_MAX)

@@ -103,9 +103,10 @@ _CORE_SIGNATURES = {
     "ap_stream_mix": [_P, _P, _I, _L, _P, _L, _I, _P, _L, _P],
     # int ap_linear_scan(q, ld_q, k, ld_k, v, ld_v, decay_channel, ld_dc, decay_head, ld_dh, decay_const, dt_bias, beta,
     #                    ld_beta, cos_sin, rot_dims, state, state_stride, seq_start, positions, state_slots, y, ld_y,
-    #                    T, nseq, heads, qk_heads, D, V, decay_mode, qk_mode, tau, unit_eps, out_scale, stream)
+    #                    T, nseq, heads, qk_heads, D, V, decay_mode, qk_mode, tau, unit_eps, out_scale, scratch, stream)
     "ap_linear_scan": [_P, _L, _P, _L, _P, _L, _P, _L, _P, _L, _P, _P, _P, _L, _P, _I, _P, _L, _P, _P, _P, _P, _L,
-                       _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _P],
+                       _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _P, _P],
+    "ap_linear_scan_block": [_I, _I, _I, _I, _I, _I],
     # int ap_head_norm_gate(y, ld_y, gate, ld_g, w, eps, out_scale, act, out, out_dtype, T, heads, V, stream)
     "ap_head_norm_gate": [_P, _L, _P, _L, _P, _F, _F, _I, _P, _I, _I, _I, _I, _P],
     # int ap_stream_norm(x, rows, R, delta, S, slice_stride, slice_bias, slice_w, slice_eps, slice_scale, out_w, mix,

@@ -30,7 +30,7 @@ def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, y: torch.Tens
                 decay_head: Optional[torch.Tensor] = None, decay_const: Optional[torch.Tensor] = None,
                 dt_bias: Optional[torch.Tensor] = None, beta: Optional[torch.Tensor] = None,
                 qk: Optional[str] = None, cos_sin: Optional[torch.Tensor] = None, unit_eps: float = 0.0,
-                out_scale: float = 1.0) -> None:
+                out_scale: float = 1.0, workspace=None) -> None:
     """Linear attention as a recurrence over each sequence's rows, all 32-bit:
     ``S = diag(a_t) S + k_t u_t^T``, ``y_t = S^T q_t * out_scale`` with a state ``[key_dim, value_dim]`` per head.
 
@@ -46,7 +46,10 @@ def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, y: torch.Tens
     ``state [slots, heads, key_dim, value_dim]`` may be a strided view of the slots' rows; a sequence whose first
     row has position 0 starts from zero.  ``q``, ``k``, ``v``, ``decay_channel``, ``decay_head`` and ``beta`` are
     scratch: a pass before the recurrence turns them into what it reads (rotated, unit or activated vectors, decays,
-    gates) in place."""
+    gates) in place.
+
+    With ``workspace`` (where the buffer between its two kernels comes from) a step whose sequences bring several rows
+    runs eight tokens at a time; without it, token after token."""
     T = y.shape[0]
     if decay not in DECAY_MODES or qk not in QK_MODES:
         raise KernelError(f"linear_scan: decay {decay!r} or qk {qk!r} is not known")
@@ -81,12 +84,18 @@ def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, y: torch.Tens
                           f"contiguous heads")
     for t, n in ((seq_start, "seq_start"), (positions, "positions"), (state_slots, "state_slots")):
         _check(t, n, torch.int32, 1)
-    call(core(), "ap_linear_scan", qp, ldq, kp, ldk, vp, ldv, dcp, dcl, dhp, dhl,
+    lib, scratch = core(), 0
+    if workspace is not None:
+        block = int(lib.ap_linear_scan_block(T, int(num_seqs), int(heads), int(key_dim), int(value_dim), DECAY_MODES[decay]))
+        if block > 0:
+            blocks = (T // 8 + int(num_seqs)) * int(heads)
+            scratch = workspace.get("linear_scan.blocks", (blocks * block,), torch.float32).data_ptr()
+    call(lib, "ap_linear_scan", qp, ldq, kp, ldk, vp, ldv, dcp, dcl, dhp, dhl,
          decay_const.data_ptr() if decay_const is not None else 0, dt_bias.data_ptr() if dt_bias is not None else 0,
          bp, bl, cos_sin.data_ptr() if rot else 0, rot, state.data_ptr(), state.stride(0), seq_start.data_ptr(),
          positions.data_ptr(), state_slots.data_ptr(), yp, ldy, T, int(num_seqs), int(heads), int(qk_heads),
          int(key_dim), int(value_dim), DECAY_MODES[decay], QK_MODES[qk], float(tau), float(unit_eps),
-         float(out_scale), stream_handle())
+         float(out_scale), scratch, stream_handle())
 
 
 def head_norm_gate(y: torch.Tensor, gate: torch.Tensor, weight: Optional[torch.Tensor], eps: float,

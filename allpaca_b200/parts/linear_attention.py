@@ -253,7 +253,7 @@ class LinearRecurrence(Mixer):
                         decay_const=self.decay_const, dt_bias=self.dt_bias,
                         beta=proj[:, c["b"]:c["b"] + self.heads] if self.delta_rule else None, qk=self.qk,
                         cos_sin=self.position.rotation_for(step)[0] if self.position is not None else None,
-                        unit_eps=self.unit_eps, out_scale=self.read_scale)
+                        unit_eps=self.unit_eps, out_scale=self.read_scale, workspace=ws)
         gated = ws.get("linrec.gated", (T, self.v_size), self.env.dtype)
         heads, V = (1, self.v_size) if self.norm_over == "row" else (self.heads, self.V)
         ops.head_norm_gate(y, gate, self.norm_w, self.norm_eps, gated, heads, V, out_scale=self.output_scale,

@@ -232,16 +232,21 @@ def plain_read(kind, t, H, G, D, V, consts, rot=None, first=0):
                                           ("channel", 5, 5, 8, 12), ("channel", 6, 6, 48, 32), ("channel", 2, 2, 40, 24),
                                           ("channel", 1, 1, 130, 7), ("head_token", 3, 1, 16, 24),
                                           ("head_token", 4, 2, 32, 32), ("head_token", 2, 2, 12, 6),
-                                          ("head_token", 8, 2, 128, 64)])
-def test_recurrences_carried_over_portions_and_slots(kind, H, G, D, V):
+                                          ("head_token", 8, 2, 128, 64), ("head_token", 1, 1, 300, 40),
+                                          ("head", 2, 2, 3, 5), ("channel", 40, 40, 16, 64)])
+@pytest.mark.parametrize("blocks", [False, True])
+def test_recurrences_carried_over_portions_and_slots(kind, H, G, D, V, blocks):
     """Two sequences whose portions share steps (a single row beside a long portion, portions of two rows), on
-    slots that held something else before; then a slot that changes hands."""
+    slots that held something else before; then a slot that changes hands.  Token after token, and four tokens at a
+    time where the portions are long enough."""
     from allpaca_b200 import ops
     g = torch.Generator().manual_seed(H * 10 + D)
     rot = {"base": 300.0, "dims": D - D % 2 if D < 20 else 16}
     consts = {"decay": torch.tensor([0.9, 0.97, 0.995, 1.0][:H] + [0.99] * max(H - 4, 0)), "tau": 4.0,
               "A_log": torch.log(0.05 + 0.5 * torch.rand(H, generator=g)), "dt_bias": torch.randn(H, generator=g) - 0.5}
     state = torch.full((2, H, D, V), float("nan"), device=DEV)
+    from allpaca_b200.parts import Workspace
+    ws = Workspace(torch.device(DEV)) if blocks else None
 
     def run(parts):
         """parts: (tensors, first position, slot) per sequence of the step."""
@@ -263,7 +268,7 @@ def test_recurrences_carried_over_portions_and_slots(kind, H, G, D, V):
             kw = dict(decay_head=cat["a"], decay_const=consts["A_log"].to(DEV), dt_bias=consts["dt_bias"].to(DEV),
                       beta=cat["b"], qk="unit", unit_eps=1e-6, out_scale=D ** -0.5)
         ops.linear_scan(cat["q"], cat["k"], cat["v"], y, state, i32(starts), i32(positions), i32([p[2] for p in parts]),
-                        len(parts), H, G, D, V, kind, **kw)
+                        len(parts), H, G, D, V, kind, workspace=ws, **kw)
         return [y[starts[j]:starts[j + 1]].cpu() for j in range(len(parts))]
 
     def cut(t, a, b):
@@ -295,14 +300,15 @@ def test_a_state_that_forgets_nothing_keeps_the_first_token():
     q[-1, 0] = 1.0                                     # the last row asks for coordinate 0
     g = torch.Generator().manual_seed(1)
     v = torch.randn(n, V, generator=g)
-    for decay in (1.0, 0.995):
+    from allpaca_b200.parts import Workspace
+    for decay, ws in ((1.0, None), (0.995, None), (1.0, Workspace(torch.device(DEV))), (0.995, Workspace(torch.device(DEV)))):
         state = torch.full((1, 1, D, V), float("nan"), device=DEV)
         at, got = 0, []
         for m in [1, 2, 64, 1, 1, 333, 2, 100, 96]:
             y = torch.empty(m, V, device=DEV)
             ops.linear_scan(q[at:at + m].to(DEV), k[at:at + m].to(DEV), v[at:at + m].to(DEV), y, state, i32([0, m]),
                             i32(list(range(at, at + m))), i32([0]), 1, 1, 1, D, V, "head",
-                            decay_const=torch.tensor([decay], device=DEV))
+                            decay_const=torch.tensor([decay], device=DEV), workspace=ws)
             got.append(y.cpu())
             at += m
         assert at == n

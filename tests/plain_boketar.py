@@ -6,6 +6,7 @@ checkpoint name.  Every function takes whole sequences ``[T, ...]`` of ONE reque
 """
 from __future__ import annotations
 
+import contextlib
 import math
 from typing import Dict, List, Optional
 
@@ -15,8 +16,26 @@ F64 = torch.float64
 UNIT_EPS = 1e-6                # under the root where the delta rule makes queries and keys unit vectors
 
 
+_ROUND: List[Optional[torch.dtype]] = [None]
+
+
+@contextlib.contextmanager
+def rounded(dtype):
+    """Within: what an engine of that storage type rounds is rounded (the inputs of products, queries, keys and values), all
+    else stays exact.  How far this moves the logits of a model says how sharply such an engine can be judged on it."""
+    _ROUND[0] = dtype
+    try:
+        yield
+    finally:
+        _ROUND[0] = None
+
+
+def stored(x):
+    return x if _ROUND[0] is None else x.to(_ROUND[0]).to(F64)
+
+
 def lin(W, name, x, bias=False):
-    y = x @ W[name].T
+    y = stored(x) @ W[name].T
     return y + W[name + ".b"] if bias else y
 
 
@@ -80,6 +99,7 @@ def rotate(x, rot, positions):
 def attend(q, k, v, scale, window, sink):
     """``q [T, H, D]``, ``k [T, G, D]``, ``v [T, G, V]``: row i over the keys ``i - window + 1 .. i`` (None: all up to
     i); the softmax's denominator also holds ``exp(sink[h])``, to which no value belongs (None: no sink)."""
+    q, k, v = stored(q), stored(k), stored(v)
     T, H, _ = q.shape
     G = k.shape[1]
     pos = torch.arange(T)
@@ -137,7 +157,7 @@ def unit(x):
 def channel_decay(W, p, m, h):
     """One decay per head and key channel: ``exp(-exp(A_log[head]) softplus(W_a2 W_a1 h + dt_bias))``, [T, H, D]."""
     H, D = int(m["heads"]), int(m["dim"])
-    z = lin(W, p + "a1", h) @ W[p + "a2"].T + W[p + "dt_bias"]
+    z = lin(W, p + "a2", lin(W, p + "a1", h)) + W[p + "dt_bias"]
     z = torch.nn.functional.softplus(z).reshape(-1, H, D)
     return torch.exp(-torch.exp(W[p + "A_log"])[None, :, None] * z)
 
@@ -166,7 +186,7 @@ def channel_delta(W, p, m, h, eps):
     k = silu(short_conv(lin(W, p + "k", h), W[p + "k.conv"])).reshape(T, G, D)
     v = silu(short_conv(lin(W, p + "v", h), W[p + "v.conv"])).reshape(T, H, V)
     o = delta_recurrence(unit(q) * D ** -0.5, unit(k), v, channel_decay(W, p, m, h), torch.sigmoid(lin(W, p + "b", h)))
-    gate = torch.sigmoid(lin(W, p + "g1", h) @ W[p + "g2"].T)
+    gate = torch.sigmoid(lin(W, p + "g2", lin(W, p + "g1", h)))
     o = (rms(o, eps) * W[p + "norm"]).reshape(T, H * V) * gate
     return lin(W, p + "o", o)
 
@@ -214,7 +234,7 @@ def forward(W, cfg, tokens, streams: Optional[List[torch.Tensor]] = None) -> tor
         xs = layer(W, cfg, i, xs)
         if streams is not None:
             streams.append(xs)
-    return norm(xs.sum(1), W["final.norm"], float(cfg["norm"]["eps"])) @ W["head"].T
+    return lin(W, "head", norm(xs.sum(1), W["final.norm"], float(cfg["norm"]["eps"])))
 
 
 def greedy(W, cfg, prompt, count: int) -> List[int]:

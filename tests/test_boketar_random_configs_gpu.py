@@ -1,10 +1,15 @@
 """Boketar configurations drawn from a seed: one to six layers of either kind in any order, with and without a
 feed-forward, 1 to 8 streams, 1 to 12 heads, head sizes that are and are not multiples of 4, rotations of 2 coordinates up
 to the whole head, windows of 1 to 300, convolutions of 1 to 9 taps, narrow pairs of 1 to 33, pages of 4 to 64.  Every
-configuration runs whole, in portions and token by token, in 32-bit and in bfloat16, against the plain implementation."""
+configuration runs whole, in portions and token by token, in 32-bit and in bfloat16, against the plain implementation.
+
+How far bfloat16's rounding moves the logits differs from draw to draw by a factor of ten (small widths, many layers, an
+embedding that weighs little beside them), so each draw is judged by its own measure: twice the largest row error that the
+plain implementation shows when it rounds what the engine stores."""
 import random
 
 import pytest
+import torch
 
 import boketar_configs as bc
 import helpers
@@ -48,10 +53,14 @@ def test_a_drawn_configuration(tmp_path, seed, dtype):
     seqs = {k: helpers.random_tokens(n, config["vocab"], 10 * seed + k) for k, n in enumerate([r.randint(40, 90), 1, 19])}
     want = {k: plain.forward(weights, config, t) for k, t in seqs.items()}
     runner = make_runner(tmp_path, dtype, 256, page_size=r.choice([4, 8, 16, 64]), max_seqs=3)
-    tally = Tally()
+    tally, tol = Tally(), TOL[dtype]
+    if dtype == "bfloat16":
+        with plain.rounded(torch.bfloat16):
+            off = plain.forward(weights, config, seqs[0]) - want[0]
+        tol = 2.0 * float((off ** 2).mean(-1).sqrt().max() / (want[0] ** 2).mean().sqrt())
     # whole; then two requests side by side in portions of any size and single rows
     for k, toks in seqs.items():
-        check(runner.step([BatchEntry(("w", k), toks, list(range(len(toks))))]), want[k], TOL[dtype], (seed, "whole", k), tally)
+        check(runner.step([BatchEntry(("w", k), toks, list(range(len(toks))))]), want[k], tol, (seed, "whole", k), tally)
         runner.finish(("w", k))
     at = {0: 0, 2: 0}
     while any(at[k] < len(seqs[k]) for k in at):
@@ -65,7 +74,7 @@ def test_a_drawn_configuration(tmp_path, seed, dtype):
         logits = runner.step(entries)
         row = 0
         for k, a, n in rows:
-            check(logits[row:row + n], want[k][a:a + n], TOL[dtype], (seed, "portion", k, a, n), tally)
+            check(logits[row:row + n], want[k][a:a + n], tol, (seed, "portion", k, a, n), tally)
             row += n
     tally.finish((seed, dtype))
     runner.finish(0)

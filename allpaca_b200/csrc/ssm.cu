@@ -86,22 +86,29 @@ causal_conv_kernel(const float* __restrict__ in, long long ld_in, int col0, cons
             for (int j = 0; j < TAPS; ++j) ww[j][i] = w[(size_t)(c + i) * TAPS + j];
 #pragma unroll
         for (int j = 0; j + 1 < TAPS; ++j) input(r0 - (TAPS - 1) + j, win[j]);
-#pragma unroll 4
-        for (int r = r0; r < r0 + rows; ++r) {
-            conv_load<VEC>(src + (size_t)(a + r) * ld_in, ib, win[TAPS - 1]);
-            float v[VEC];
+        for (int rr = r0; rr < r0 + rows; rr += 4) {
+            float next[4][VEC];                               // four rows on their way together
 #pragma unroll
-            for (int i = 0; i < VEC; ++i) {
-                v[i] = ob[i];
+            for (int k = 0; k < 4; ++k)
+                if (rr + k < r0 + rows) conv_load<VEC>(src + (size_t)(a + rr + k) * ld_in, ib, next[k]);
 #pragma unroll
-                for (int j = 0; j < TAPS; ++j) v[i] = fmaf(ww[j][i], win[j][i], v[i]);
-                if (act == CONV_ACT_SILU) v[i] = ssm_silu(v[i]);
+            for (int k = 0; k < 4; ++k) {
+                if (rr + k >= r0 + rows) break;
+                float v[VEC];
 #pragma unroll
-                for (int j = 0; j + 1 < TAPS; ++j) win[j][i] = win[j + 1][i];
+                for (int i = 0; i < VEC; ++i) {
+                    win[TAPS - 1][i] = next[k][i];
+                    v[i] = ob[i];
+#pragma unroll
+                    for (int j = 0; j < TAPS; ++j) v[i] = fmaf(ww[j][i], win[j][i], v[i]);
+                    if (act == CONV_ACT_SILU) v[i] = ssm_silu(v[i]);
+#pragma unroll
+                    for (int j = 0; j + 1 < TAPS; ++j) win[j][i] = win[j + 1][i];
+                }
+                float* o = out + (size_t)(a + rr + k) * C + c;
+                if constexpr (VEC == 4) *reinterpret_cast<float4*>(o) = make_float4(v[0], v[1], v[2], v[3]);
+                else o[0] = v[0];
             }
-            float* o = out + (size_t)(a + r) * C + c;
-            if constexpr (VEC == 4) *reinterpret_cast<float4*>(o) = make_float4(v[0], v[1], v[2], v[3]);
-            else o[0] = v[0];
         }
     } else {
         for (int r = r0; r < r0 + rows; ++r) {
@@ -137,10 +144,10 @@ AP_EXPORT int ap_causal_conv(const float* in, long long ld_in, int col0, const f
     AP_REQUIRE(act == CONV_ACT_NONE || act == CONV_ACT_SILU, "causal_conv: activation %d is not known", act);
     AP_REQUIRE(taps == 1 || state != nullptr, "causal_conv: a convolution over several tokens needs its state");
     if (T == 0 || nseq == 0) return AP_OK;
-    const int run = taps - 1 > CONV_ROWS ? taps - 1 : CONV_ROWS;
     const bool vec = C % 4 == 0 && col0 % 4 == 0 && ld_in % 4 == 0 && ((((uintptr_t)in) | ((uintptr_t)out)) & 15) == 0 &&
                      taps <= 6;
     const int per = CONV_THREADS * (vec ? 4 : 1);
+    const int run = taps - 1 > CONV_ROWS ? taps - 1 : CONV_ROWS;
     const dim3 grid((unsigned)(T / run + nseq), (unsigned)((C + per - 1) / per));
 #define LAUNCH(N, V)                                                                                                \
     AP_CHECK_PDL_LAUNCH("causal_conv", ap_launch_pdl(causal_conv_kernel<N, V>, grid, dim3(CONV_THREADS), 0, stream, in, \

@@ -22,7 +22,7 @@ _ROUND: List[Optional[torch.dtype]] = [None]
 @contextlib.contextmanager
 def rounded(dtype):
     """Within: what an engine of that storage type rounds is rounded (the inputs of products, queries, keys and values), all
-    else stays exact.  How far this moves the logits of a model says how sharply such an engine can be judged on it."""
+    else stays exact.  How far this moves the logits of a model says how closely such an engine can follow it."""
     _ROUND[0] = dtype
     try:
         yield

@@ -4,7 +4,7 @@ to the whole head, windows of 1 to 300, convolutions of 1 to 9 taps, narrow pair
 configuration runs whole, in portions and token by token, in 32-bit and in bfloat16, against the plain implementation.
 
 How far bfloat16's rounding moves the logits differs from draw to draw by a factor of ten (small widths, many layers, an
-embedding that weighs little beside them), so each draw is judged by its own measure: twice the largest row error that the
+embedding that weighs little beside them), so each draw has its own tolerance: twice the largest row error that the
 plain implementation shows when it rounds what the engine stores."""
 import random
 

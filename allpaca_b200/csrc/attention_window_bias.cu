@@ -146,7 +146,9 @@ AP_EXPORT int ap_qk_norm_store(const void* in, int in_dtype, long long ld_in, vo
                                int normalise, float temp_coef, int temp_every, const float* qw, const float* kw,
                                const float* bias, const float* cos_sin, int rot_dims, int pairing,
                                float value_scale, cudaStream_t stream) {
-    AP_REQUIRE(T >= 0 && nh > 0 && nkv > 0 && D > 0 && VD > 0 && D <= MAX_HEAD && VD <= MAX_HEAD,
+    // without pages only the queries are made ready, and the projection need not hold keys and values
+    if (cache == nullptr) nkv = 0;
+    AP_REQUIRE(T >= 0 && nh > 0 && nkv >= (cache ? 1 : 0) && D > 0 && VD > 0 && D <= MAX_HEAD && VD <= MAX_HEAD,
                "qk_norm_store: bad sizes T=%d heads=%d/%d sizes %d/%d (at most %d)", T, nh, nkv, D, VD, MAX_HEAD);
     AP_REQUIRE(cache == nullptr || (token_seq && block_table && max_blocks > 0 && P > 0),
                "qk_norm_store: storing needs token_seq and a block table");

@@ -7,9 +7,13 @@
 //   decay a_t   one fixed number per head (DECAY_HEAD_CONST: retention);
 //               one number per head and token, exp(-exp(A_log[h]) * softplus(raw + dt_bias[h])) (DECAY_HEAD_TOKEN);
 //               one number per key channel and token, sigmoid(z)^(1/tau) = exp(-softplus(-z) / tau) (DECAY_CHANNEL),
-//               or exp(-exp(A_log[h]) * softplus(z + dt_bias[h, channel])) (DECAY_CHANNEL_TOKEN)
-//   write u_t   the value v_t; or, with the delta rule, beta_t (v_t - S^T k_t) with S already decayed and
-//               beta_t = sigmoid(raw), so that the read-out sees the corrected state
+//               or exp(-exp(A_log[h]) * softplus(z + dt_bias[h, channel])) (DECAY_CHANNEL_TOKEN);
+//               or one number per head and token that another kernel has worked out (DECAY_HEAD_READY)
+//   write u_t   the value v_t, or b_t v_t with a number per head and token that another kernel has worked out; or, with
+//               the delta rule, beta_t (v_t - S^T k_t) with S already decayed and beta_t = sigmoid(raw), so that the
+//               read-out sees the corrected state
+//   unit column the values may have one more column that is always 1: the state's last column then is the sum of
+//               the keys themselves under the same decays and gates, and its read-out their product with the query
 //   q, k        as projected (QK_PLAIN); the first rot_dims coordinates of every head turned by the step's
 //               cosine/sine table, coordinate i with i + rot_dims/2 (QK_ROTATE); or made unit vectors,
 //               x / sqrt(sum x^2 + unit_eps) (QK_UNIT); or, like the values, under SiLU (QKV_SILU).  Several value
@@ -34,10 +38,14 @@
 #define DECAY_HEAD_TOKEN 1
 #define DECAY_CHANNEL 2
 #define DECAY_CHANNEL_TOKEN 3
+#define DECAY_HEAD_READY 4
 #define QK_PLAIN 0
 #define QK_ROTATE 1
 #define QK_UNIT 2
 #define QKV_SILU 3
+
+// whether every key channel has a decay of its own
+__host__ __device__ constexpr bool la_per_channel(int mode) { return mode == DECAY_CHANNEL || mode == DECAY_CHANNEL_TOKEN; }
 
 __device__ __forceinline__ float la_softplus(float v) { return v > 20.0f ? v : log1pf(expf(v)); }
 __device__ __forceinline__ float la_silu(float v) { return v / (1.0f + expf(-v)); }
@@ -55,15 +63,17 @@ struct LaScanArgs {
     float* k; long long ld_k;
     float* v; long long ld_v;                  // head h of row t: v[t * ld_v + h * V + c]; QKV_SILU: in place
     float* decay_channel; long long ld_dc;     // DECAY_CHANNEL*: z[t * ld_dc + h * D + d], becomes the decay in place
-    float* decay_head; long long ld_dh;        // DECAY_HEAD_TOKEN: raw[t * ld_dh + h], becomes the decay in place
+    float* decay_head; long long ld_dh;        // DECAY_HEAD_TOKEN: raw[t * ld_dh + h], becomes the decay in place; DECAY_HEAD_READY: it
     const float* decay_const;                  // DECAY_HEAD_CONST: the decay [heads]; DECAY_*_TOKEN: A_log [heads]
     const float* dt_bias;                      // DECAY_HEAD_TOKEN: [heads], DECAY_CHANNEL_TOKEN: [heads * D]; or null
-    float* beta; long long ld_beta;            // raw[t * ld_beta + h], becomes sigmoid in place; null: no delta rule
+    float* beta; long long ld_beta;            // the write's gate [t * ld_beta + h], or null: it is 1
+    int delta;                                 // the delta rule (its gate comes raw and becomes sigmoid in place)
     const float* cos_sin; int rot_dims;        // QK_ROTATE: [T, rot_dims / 2, 2]
     float* state; long long state_stride;      // [slots][heads][D][V]
     const int* seq_start; const int* positions; const int* state_slots;
     float* y; long long ld_y;                  // y[t * ld_y + h * V + c]
     int T, heads, qk_heads, D, V, NP, cols, decay_mode, qk_mode, vec;
+    int VI;                                    // columns of v: V, or V - 1 where the last one is always 1
     float inv_tau, unit_eps, out_scale;
 };
 
@@ -78,8 +88,8 @@ __global__ void __launch_bounds__(128) la_prepare_kernel(const LaScanArgs A) {
     const int G = A.qk_heads, H = A.heads, D = A.D;
     const int qk_units = A.qk_mode == QK_PLAIN ? 0 : 2 * G;
     const int v_units = A.qk_mode == QKV_SILU ? H : 0;
-    const int ch_units = A.decay_mode >= DECAY_CHANNEL ? H : 0;
-    const int sc_units = (A.decay_mode == DECAY_HEAD_TOKEN || A.beta != nullptr) ? 1 : 0;
+    const int ch_units = la_per_channel(A.decay_mode) ? H : 0;
+    const int sc_units = (A.decay_mode == DECAY_HEAD_TOKEN || A.delta) ? 1 : 0;
     const int units = qk_units + v_units + ch_units + sc_units;
     const long long unit = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
     if (unit >= (long long)A.T * units) return;
@@ -129,7 +139,7 @@ __global__ void __launch_bounds__(128) la_prepare_kernel(const LaScanArgs A) {
             float* a = A.decay_head + (size_t)t * A.ld_dh + h;
             *a = expf(-expf(A.decay_const[h]) * la_softplus(*a + (A.dt_bias ? A.dt_bias[h] : 0.f)));
         }
-        if (A.beta) {
+        if (A.delta) {
             float* b = A.beta + (size_t)t * A.ld_beta + h;
             *b = 1.0f / (1.0f + expf(-*b));
         }
@@ -159,8 +169,9 @@ __global__ void __launch_bounds__(128) la_scan_kernel(const LaScanArgs A) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
     const int vcol = col0 + vl;
     const bool live = vl < ncols;
-    const bool channel = A.decay_mode >= DECAY_CHANNEL, delta = A.beta != nullptr;
-    const bool token_decay = A.decay_mode == DECAY_HEAD_TOKEN;
+    const bool channel = la_per_channel(A.decay_mode), delta = A.delta != 0, gated = A.beta != nullptr;
+    const bool token_decay = A.decay_mode == DECAY_HEAD_TOKEN || A.decay_mode == DECAY_HEAD_READY;
+    const int vcols = min(ncols, A.VI - col0);               // columns that v brings; the unit column (if it lies here) follows
     const int XS = (cols + 3) / 4 * 4, DS = PER * NP;        // a row of keys in shared memory is padded with zeros
     // one buffer: v [CHUNK][XS], k [CHUNK][DS], q [CHUNK][DS], channel decays [CHUNK][DS] (if any), decay [CHUNK], beta [CHUNK]
     const int buf_floats = LA_CHUNK * (XS + (channel ? 3 : 2) * DS) + 2 * LA_CHUNK;
@@ -172,6 +183,9 @@ __global__ void __launch_bounds__(128) la_scan_kernel(const LaScanArgs A) {
             sm[b * buf_floats + LA_CHUNK * XS + (j / pad) * DS + D + j % pad] = 0.f;
         }
     }
+    if (vcols < ncols)                                       // no copy writes it
+        for (int i = threadIdx.x; i < 2 * LA_CHUNK; i += blockDim.x)
+            sm[(i / LA_CHUNK) * buf_floats + (i % LA_CHUNK) * XS + vcols] = 1.f;
     float* st = A.state + (size_t)A.state_slots[s] * A.state_stride + (size_t)h * D * V;
     const bool fresh = A.positions[a] == 0;
     float S[PER];
@@ -194,9 +208,9 @@ __global__ void __launch_bounds__(128) la_scan_kernel(const LaScanArgs A) {
         const size_t row = (size_t)(a + t0);
         // values: eight threads to a row; keys, queries and channel decays: a warp to a row, the lanes across it
         for (int r = threadIdx.x >> 3; r < cnt; r += blockDim.x >> 3) {
-            const float* src = A.v + (row + r) * A.ld_v + (size_t)h * V + col0;
-            if (vec && ncols % 4 == 0) for (int d = (threadIdx.x & 7) * 4; d < ncols; d += 32) la_copy16(v_b + r * XS + d, src + d);
-            else for (int d = threadIdx.x & 7; d < ncols; d += 8) la_copy4(v_b + r * XS + d, src + d);
+            const float* src = A.v + (row + r) * A.ld_v + (size_t)h * A.VI + col0;
+            if (vec && vcols % 4 == 0) for (int d = (threadIdx.x & 7) * 4; d < vcols; d += 32) la_copy16(v_b + r * XS + d, src + d);
+            else for (int d = threadIdx.x & 7; d < vcols; d += 8) la_copy4(v_b + r * XS + d, src + d);
         }
         for (int r = warp; r < cnt; r += nwarps) {
             const float* ks = A.k + (row + r) * A.ld_k + (size_t)g * D;
@@ -218,7 +232,7 @@ __global__ void __launch_bounds__(128) la_scan_kernel(const LaScanArgs A) {
         }
         if ((int)threadIdx.x < cnt) {
             if (token_decay) la_copy4(sc_b + threadIdx.x, A.decay_head + (row + threadIdx.x) * A.ld_dh + h);
-            if (delta) la_copy4(sc_b + LA_CHUNK + threadIdx.x, A.beta + (row + threadIdx.x) * A.ld_beta + h);
+            if (gated) la_copy4(sc_b + LA_CHUNK + threadIdx.x, A.beta + (row + threadIdx.x) * A.ld_beta + h);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -262,6 +276,7 @@ __global__ void __launch_bounds__(128) la_scan_kernel(const LaScanArgs A) {
                 for (int i = 0; i < PER; ++i) S[i] *= dec;
             }
             float u = vv;
+            if (gated && !delta) u = sc_s[LA_CHUNK + r] * vv;
             if (delta) {
                 float d0 = 0.f, d1 = 0.f, d2 = 0.f, d3 = 0.f;
 #pragma unroll
@@ -379,7 +394,6 @@ __global__ void __launch_bounds__(128, 4) la_blocks_kernel(const LaScanArgs A, c
     float* kh = qt + LT * DS;
     float* ct = kh + LT * DS;
     float* vb = CH ? ct + DS : kh;
-    const bool delta = A.beta != nullptr;
     const int mode = A.qk_mode, half = A.rot_dims / 2;
     const float* qp = A.q + (size_t)row * A.ld_q + (size_t)g * D;
     const float* kp = A.k + (size_t)row * A.ld_k + (size_t)g * D;
@@ -390,8 +404,9 @@ __global__ void __launch_bounds__(128, 4) la_blocks_kernel(const LaScanArgs A, c
         const size_t t = (size_t)row + r;
         float b = r < cnt ? 1.f : 0.f, a = 1.f;
         if (r < cnt) {
-            if (delta) b = 1.0f / (1.0f + expf(-A.beta[t * A.ld_beta + h]));
+            if (A.beta) b = A.delta ? 1.0f / (1.0f + expf(-A.beta[t * A.ld_beta + h])) : A.beta[t * A.ld_beta + h];
             if (A.decay_mode == DECAY_HEAD_CONST) a = A.decay_const[h];
+            if (A.decay_mode == DECAY_HEAD_READY) a = A.decay_head[t * A.ld_dh + h];
             if (A.decay_mode == DECAY_HEAD_TOKEN)
                 a = expf(-expf(A.decay_const[h]) * la_softplus(A.decay_head[t * A.ld_dh + h] + (A.dt_bias ? A.dt_bias[h] : 0.f)));
         }
@@ -519,11 +534,12 @@ __global__ void __launch_bounds__(128, 4) la_blocks_kernel(const LaScanArgs A, c
         if (r == LT - 1) rec[REC_TOTAL] = upto;
     }
     for (int r = 0; r < LT; ++r) {
-        const float* vp = A.v + ((size_t)row + r) * A.ld_v + (size_t)h * V;
+        const float* vp = A.v + ((size_t)row + r) * A.ld_v + (size_t)h * A.VI;
         for (int d = threadIdx.x; d < VS; d += blockDim.x) {
-            float v = (r < cnt && d < V) ? vp[d] : 0.f;
+            float v = (r < cnt && d < A.VI) ? vp[d] : 0.f;
             if (mode == QKV_SILU) v = la_silu(v);
-            vb[r * VS + d] = delta ? beta[r] * v : v;
+            if (d >= A.VI && d < V) v = 1.f;                 // (beta is 0 beyond the last token)
+            vb[r * VS + d] = beta[r] * v;
         }
     }
 }
@@ -812,7 +828,7 @@ AP_EXPORT int ap_linear_scan_block(int T, int nseq, int heads, int D, int V, int
     if (T <= 0 || nseq <= 0 || heads <= 0 || D <= 0 || V <= 0 || !la_in_blocks(T, nseq)) return 0;
     int NP, per, cpt;
     lc_plan(nseq, heads, D, V, NP, per, cpt);
-    return REC_SIZE + (decay_mode >= DECAY_CHANNEL ? 3 * LT + 1 : 2 * LT) * per * NP + LT * ((V + 3) / 4 * 4);
+    return REC_SIZE + (la_per_channel(decay_mode) ? 3 * LT + 1 : 2 * LT) * per * NP + LT * ((V + 3) / 4 * 4);
 }
 
 typedef void (*la_chunk_fn)(const LaScanArgs, const LaBlocks, int);
@@ -830,7 +846,7 @@ static int la_run_blocks(LaScanArgs& A, int nseq, float* scratch, cudaStream_t s
     B.at = scratch;
     B.DS = per * NP;
     B.VS = (A.V + 3) / 4 * 4;
-    const bool channel = A.decay_mode >= DECAY_CHANNEL, delta = A.beta != nullptr;
+    const bool channel = la_per_channel(A.decay_mode), delta = A.delta != 0;
     const int main_floats = REC_SIZE + (channel ? 3 * LT + 1 : 2 * LT) * B.DS;
     B.size = main_floats + LT * B.VS;
     const int cols = 128 / NP * cpt;
@@ -864,8 +880,8 @@ AP_EXPORT int ap_linear_scan(float* q, long long ld_q, float* k, long long ld_k,
                              long long ld_beta, const float* cos_sin, int rot_dims, float* state,
                              long long state_stride, const int* seq_start, const int* positions,
                              const int* state_slots, float* y, long long ld_y, int T, int nseq, int heads,
-                             int qk_heads, int D, int V, int decay_mode, int qk_mode, float tau, float unit_eps,
-                             float out_scale, float* scratch, cudaStream_t stream) {
+                             int qk_heads, int D, int V, int decay_mode, int qk_mode, int delta, int unit_column, float tau,
+                             float unit_eps, float out_scale, float* scratch, cudaStream_t stream) {
     AP_REQUIRE(T >= 0 && nseq >= 0 && heads > 0 && qk_heads > 0 && heads % qk_heads == 0 && D > 0 && V > 0,
                "linear_scan: bad sizes heads=%d qk_heads=%d key=%d value=%d", heads, qk_heads, D, V);
     AP_REQUIRE(D <= LA_PER_MAX * 32, "linear_scan: keys of %d exceed %d", D, LA_PER_MAX * 32);
@@ -874,8 +890,11 @@ AP_EXPORT int ap_linear_scan(float* q, long long ld_q, float* k, long long ld_k,
     AP_REQUIRE(decay_mode == DECAY_HEAD_CONST ? decay_const != nullptr
                : decay_mode == DECAY_HEAD_TOKEN ? (decay_head != nullptr && decay_const != nullptr)
                : decay_mode == DECAY_CHANNEL ? (decay_channel != nullptr && tau > 0.f)
+               : decay_mode == DECAY_HEAD_READY ? decay_head != nullptr
                : (decay_mode == DECAY_CHANNEL_TOKEN && decay_channel != nullptr && decay_const != nullptr),
                "linear_scan: decay mode %d lacks its numbers", decay_mode);
+    AP_REQUIRE(!delta || beta != nullptr, "linear_scan: the delta rule lacks its gates");
+    AP_REQUIRE(!unit_column || (V > 1 && qk_mode != QKV_SILU), "linear_scan: a unit column goes with plain values");
     AP_REQUIRE(qk_mode == QK_PLAIN || qk_mode == QK_UNIT || qk_mode == QKV_SILU ||
                (qk_mode == QK_ROTATE && cos_sin && rot_dims > 0 && rot_dims % 2 == 0 && rot_dims <= D),
                "linear_scan: query/key mode %d with %d rotated coordinates of %d", qk_mode, rot_dims, D);
@@ -892,9 +911,10 @@ AP_EXPORT int ap_linear_scan(float* q, long long ld_q, float* k, long long ld_k,
     const dim3 grid((unsigned)nseq, (unsigned)heads, (unsigned)((V + cols - 1) / cols));
     AP_REQUIRE(heads <= 65535 && grid.z <= 65535, "linear_scan: %d heads exceed the grid", heads);
     auto aligned = [](const void* p, long long ld) { return p == nullptr || ((((uintptr_t)p) & 15) == 0 && ld % 4 == 0); };
-    const int vec = (D % 4 == 0 && V % 4 == 0 && cols % 4 == 0 && aligned(q, ld_q) && aligned(k, ld_k) &&
+    const int VI = V - (unit_column ? 1 : 0);
+    const int vec = (D % 4 == 0 && VI % 4 == 0 && cols % 4 == 0 && aligned(q, ld_q) && aligned(k, ld_k) &&
                      aligned(v, ld_v) && aligned(decay_channel, ld_dc)) ? 1 : 0;
-    const bool channel = decay_mode >= DECAY_CHANNEL;
+    const bool channel = la_per_channel(decay_mode);
     LaScanArgs A;
     A.q = q; A.ld_q = ld_q; A.k = k; A.ld_k = ld_k; A.v = v; A.ld_v = ld_v;
     A.decay_channel = decay_channel; A.ld_dc = ld_dc; A.decay_head = decay_head; A.ld_dh = ld_dh;
@@ -902,11 +922,11 @@ AP_EXPORT int ap_linear_scan(float* q, long long ld_q, float* k, long long ld_k,
     A.cos_sin = cos_sin; A.rot_dims = rot_dims; A.state = state; A.state_stride = state_stride;
     A.seq_start = seq_start; A.positions = positions; A.state_slots = state_slots; A.y = y; A.ld_y = ld_y;
     A.T = T; A.heads = heads; A.qk_heads = qk_heads; A.D = D; A.V = V; A.NP = NP; A.cols = cols;
-    A.decay_mode = decay_mode; A.qk_mode = qk_mode; A.vec = vec;
+    A.decay_mode = decay_mode; A.qk_mode = qk_mode; A.vec = vec; A.delta = delta ? 1 : 0; A.VI = VI;
     A.inv_tau = decay_mode == DECAY_CHANNEL ? 1.0f / tau : 0.f; A.unit_eps = unit_eps; A.out_scale = out_scale;
     if (scratch != nullptr && la_in_blocks(T, nseq)) return la_run_blocks(A, nseq, scratch, stream);
     const int units = (qk_mode == QK_PLAIN ? 0 : 2 * qk_heads) + (qk_mode == QKV_SILU ? heads : 0) + (channel ? heads : 0) +
-                      ((decay_mode == DECAY_HEAD_TOKEN || beta != nullptr) ? 1 : 0);
+                      ((decay_mode == DECAY_HEAD_TOKEN || delta) ? 1 : 0);
     if (units > 0) {
         const long long blocks = ((long long)T * units + 3) / 4;
         AP_CHECK_PDL_LAUNCH("linear_scan (rows made ready)",
@@ -930,18 +950,115 @@ AP_EXPORT int ap_linear_scan(float* q, long long ld_q, float* k, long long ld_k,
     return AP_OK;
 }
 
+// ---- exponential gates under a running maximum ------------------------------------------------
+// A head's log input gate i = cap tanh((raw_i + b_i) / cap) and log forget gate f = logsigmoid(cap tanh((raw_f + b_f) / cap))
+// may differ by many orders of magnitude from token to token, so the state is kept as exp(-m) times what the gates
+// alone would make of it, with m a running maximum that a request carries from step to step (0 at its start):
+//
+//   m_t = max(f_t + m_{t-1}, i_t)     decay_t = exp(f_t + m_{t-1} - m_t)     write_t = exp(i_t - m_t)     floor_t = exp(-m_t)
+//
+// Decay and write replace the raw numbers in place (both are at most 1); floor is what 1 has become under the same scale.
+// One CTA per (head, sequence).  A token is the map m -> max(f + m, i); maps compose (sums of f, a maximum), so a thread
+// composes XG_PER tokens, the threads' maps meet in a scan, and each thread then walks its tokens from the m it starts at.
+#define XG_PER 4
+#define XG_THREADS 256
+
+__device__ __forceinline__ float la_logsigmoid(float v) { return fminf(v, 0.f) - log1pf(expf(-fabsf(v))); }
+
+__global__ void __launch_bounds__(XG_THREADS)
+exp_gates_kernel(float* __restrict__ gi, float* __restrict__ gf, long long ld, const float* __restrict__ bi,
+                 const float* __restrict__ bf, float cap, float* __restrict__ state, long long state_stride,
+                 const int* __restrict__ seq_start, const int* __restrict__ positions,
+                 const int* __restrict__ state_slots, float* __restrict__ floor_out, int heads) {
+    __shared__ float sum_s[XG_THREADS / 32], top_s[XG_THREADS / 32];
+    ap_pdl_trigger();
+    ap_pdl_wait();
+    const int h = blockIdx.x, s = blockIdx.y;
+    const int a = seq_start[s], n = seq_start[s + 1] - a;
+    if (n <= 0) return;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
+    float* mine = state + (size_t)state_slots[s] * state_stride + h;
+    float m0 = positions[a] == 0 ? 0.f : *mine;
+    const float add_i = bi ? bi[h] : 0.f, add_f = bf ? bf[h] : 0.f;
+    for (int t0 = 0; t0 < n; t0 += XG_PER * blockDim.x) {
+        float in[XG_PER], fo[XG_PER];
+        float sum = 0.f, top = -INFINITY;                    // this thread's map: m -> max(sum + m, top)
+#pragma unroll
+        for (int j = 0; j < XG_PER; ++j) {
+            const int t = t0 + threadIdx.x * XG_PER + j;
+            in[j] = -INFINITY;                               // beyond the end: m stays
+            fo[j] = 0.f;
+            if (t < n) {
+                in[j] = cap * tanhf((gi[(size_t)(a + t) * ld + h] + add_i) / cap);
+                fo[j] = la_logsigmoid(cap * tanhf((gf[(size_t)(a + t) * ld + h] + add_f) / cap));
+            }
+            sum += fo[j];
+            top = fmaxf(fo[j] + top, in[j]);
+        }
+        // scan over the lanes: the map of everything up to and with this thread
+        float psum = sum, ptop = top;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const float bs = __shfl_up_sync(0xffffffffu, psum, o), bt = __shfl_up_sync(0xffffffffu, ptop, o);
+            if (lane >= o) {
+                ptop = fmaxf(psum + bt, ptop);
+                psum += bs;
+            }
+        }
+        if (lane == 31) { sum_s[warp] = psum; top_s[warp] = ptop; }
+        __syncthreads();
+        float m = m0;                                        // the m before this warp's first token, and after the last
+        for (int w = 0; w < nwarps; ++w) {
+            if (w == warp) m = m0;
+            m0 = fmaxf(sum_s[w] + m0, top_s[w]);
+        }
+        const float es = __shfl_up_sync(0xffffffffu, psum, 1), et = __shfl_up_sync(0xffffffffu, ptop, 1);
+        if (lane > 0) m = fmaxf(es + m, et);
+        float last = m;
+#pragma unroll
+        for (int j = 0; j < XG_PER; ++j) {
+            const int t = t0 + threadIdx.x * XG_PER + j;
+            if (t >= n) break;
+            const float next = fmaxf(fo[j] + last, in[j]);
+            gf[(size_t)(a + t) * ld + h] = expf(fo[j] + last - next);
+            gi[(size_t)(a + t) * ld + h] = expf(in[j] - next);
+            floor_out[(size_t)(a + t) * heads + h] = expf(-next);
+            last = next;
+        }
+        __syncthreads();
+    }
+    if (threadIdx.x == 0) *mine = m0;
+}
+
+AP_EXPORT int ap_exp_gates(float* gi, float* gf, long long ld, const float* bi, const float* bf, float cap, float* state,
+                           long long state_stride, const int* seq_start, const int* positions, const int* state_slots,
+                           float* floor_out, int T, int nseq, int heads, cudaStream_t stream) {
+    AP_REQUIRE(T >= 0 && nseq >= 0 && heads > 0 && ld >= heads && cap > 0.f && state_stride >= heads && gi && gf && state &&
+               floor_out, "exp_gates: bad arguments heads=%d cap=%f", heads, (double)cap);
+    AP_REQUIRE(nseq <= 65535, "exp_gates: %d sequences exceed the grid", nseq);
+    if (T == 0 || nseq == 0) return AP_OK;
+    int threads = 32;                                        // as many as the longest portion could fill
+    while (threads < XG_THREADS && threads * XG_PER < T - nseq + 1) threads *= 2;
+    AP_CHECK_PDL_LAUNCH("exp_gates", ap_launch_pdl(exp_gates_kernel, dim3((unsigned)heads, (unsigned)nseq), dim3((unsigned)threads), 0,
+                                                   stream, gi, gf, ld, bi, bf, cap, state, state_stride, seq_start, positions,
+                                                   state_slots, floor_out, heads));
+    return AP_OK;
+}
+
 // ---- a head's read-out: RMS norm, gate, constant ------------------------------------------
-// y: [T, ld_y] 32-bit, head h at column h * V; gate: [T, ld_g] 32-bit raw, same layout; `threads` (a warp, or a CTA
-// where the heads are long: a norm over all heads together is one head of their whole width) per (row, head).
+// y: [T, ld_y] 32-bit, head h at column h * hs; gate: [T, ld_g] 32-bit raw, head h at column h * V; `threads` (a warp, or a
+// CTA where the heads are long: a norm over all heads together is one head of their whole width) per (row, head).
+// With `floor` [T, heads] (hs is V + 1 then) the head's numbers are first divided by max(|number V|, floor) + floor_eps.
+// The weight has V numbers that the heads share, or (`own_weights`) V for each head.
 #define GATE_SILU 0
 #define GATE_SIGMOID 1
 #define HNG_THREADS 128
 
 template <typename TO, bool WHOLE_CTA>
 __global__ void __launch_bounds__(HNG_THREADS)
-head_norm_gate_kernel(const float* __restrict__ y, long long ld_y, const float* __restrict__ gate, long long ld_g,
-                      const float* __restrict__ w, float eps, float out_scale, int act, TO* __restrict__ out, int T,
-                      int heads, int V) {
+head_norm_gate_kernel(const float* __restrict__ y, long long ld_y, int hs, const float* __restrict__ floor_in,
+                      float floor_eps, const float* __restrict__ gate, long long ld_g, const float* __restrict__ w,
+                      int own_weights, float eps, float out_scale, int act, TO* __restrict__ out, int T, int heads, int V) {
     __shared__ float scratch[32];
     ap_pdl_trigger();
     ap_pdl_wait();
@@ -949,12 +1066,17 @@ head_norm_gate_kernel(const float* __restrict__ y, long long ld_y, const float* 
     if (unit >= (long long)T * heads) return;                // (a whole CTA always has its unit)
     const int first = WHOLE_CTA ? threadIdx.x : (threadIdx.x & 31), stride = WHOLE_CTA ? HNG_THREADS : 32;
     const int t = (int)(unit / heads), h = (int)(unit % heads);
-    const float* yr = y + (size_t)t * ld_y + (size_t)h * V;
+    const float* yr = y + (size_t)t * ld_y + (size_t)h * hs;
     const float* gr = gate + (size_t)t * ld_g + (size_t)h * V;
+    if (w && own_weights) w += (size_t)h * V;
+    const float pre = floor_in ? 1.0f / (fmaxf(fabsf(yr[V]), floor_in[(size_t)t * heads + h]) + floor_eps) : 1.0f;
     float ss = 0.f;
-    for (int i = first; i < V; i += stride) ss = fmaf(yr[i], yr[i], ss);
+    for (int i = first; i < V; i += stride) {
+        const float v = yr[i] * pre;
+        ss = fmaf(v, v, ss);
+    }
     ss = WHOLE_CTA ? ap_block_sum(ss, scratch) : ap_warp_sum(ss);
-    const float inv = out_scale / sqrtf(ss / (float)V + eps);
+    const float inv = pre * (out_scale / sqrtf(ss / (float)V + eps));
     TO* o = out + ((size_t)t * heads + h) * V;
     for (int i = first; i < V; i += stride) {
         const float s = 1.0f / (1.0f + expf(-gr[i]));
@@ -962,11 +1084,12 @@ head_norm_gate_kernel(const float* __restrict__ y, long long ld_y, const float* 
     }
 }
 
-AP_EXPORT int ap_head_norm_gate(const float* y, long long ld_y, const float* gate, long long ld_g, const float* w,
-                                float eps, float out_scale, int act, void* out, int out_dtype, int T, int heads, int V,
+AP_EXPORT int ap_head_norm_gate(const float* y, long long ld_y, int hs, const float* floor_in, float floor_eps,
+                                const float* gate, long long ld_g, const float* w, int own_weights, float eps,
+                                float out_scale, int act, void* out, int out_dtype, int T, int heads, int V,
                                 cudaStream_t stream) {
-    AP_REQUIRE(T >= 0 && heads > 0 && V > 0 && ld_y >= (long long)heads * V && ld_g >= (long long)heads * V,
-               "head_norm_gate: bad sizes heads=%d value=%d", heads, V);
+    AP_REQUIRE(T >= 0 && heads > 0 && V > 0 && hs >= V + (floor_in ? 1 : 0) && ld_y >= (long long)heads * hs &&
+               ld_g >= (long long)heads * V, "head_norm_gate: bad sizes heads=%d value=%d stride=%d", heads, V, hs);
     AP_REQUIRE(act == GATE_SILU || act == GATE_SIGMOID, "head_norm_gate: gate %d is not known", act);
     if (T == 0) return AP_OK;
     const bool whole = V > 256;
@@ -974,7 +1097,8 @@ AP_EXPORT int ap_head_norm_gate(const float* y, long long ld_y, const float* gat
     const dim3 grid((unsigned)((units + per - 1) / per));
 #define LAUNCH(TO, WHOLE)                                                                                           \
     AP_CHECK_PDL_LAUNCH("head_norm_gate", ap_launch_pdl(head_norm_gate_kernel<TO, WHOLE>, grid, dim3(HNG_THREADS), 0, stream, \
-                                                        y, ld_y, gate, ld_g, w, eps, out_scale, act, (TO*)out, T, heads, V))
+                                                        y, ld_y, hs, floor_in, floor_eps, gate, ld_g, w, own_weights, eps, \
+                                                        out_scale, act, (TO*)out, T, heads, V))
     if (out_dtype == AP_F32) { if (whole) LAUNCH(float, true); else LAUNCH(float, false); }
     else if (out_dtype == AP_BF16) { if (whole) LAUNCH(bf16, true); else LAUNCH(bf16, false); }
     else AP_REQUIRE(false, "head_norm_gate: unknown dtype %d", out_dtype);

@@ -3,19 +3,26 @@
 //   moe_route      per row: the `top` experts with the largest router logits (ties: the lower
 //                  index), shares = exp(z_e) / sum over the selected exp(z_s); all 32-bit.  Or
 //                  (ROUTE_SOFTMAX_ALL) scores s = softmax(z) over all experts, the `top` largest
-//                  s + bias chosen, shares = the chosen s divided by their sum.  Experts from
+//                  s + bias chosen, shares = the chosen s divided by their sum (ROUTE_SOFTMAX_SCORES:
+//                  as they are).  The choice may be among the experts of the best `keep` of `groups`
+//                  equal groups of neighbours only (a group counts as its best expert); shares may
+//                  be multiplied by a constant.  Experts from
 //                  `real` on are identity experts: no weights, their result is the row's input
 //   moe_sort       (row, choice) pairs grouped by expert: a permutation, every pair's place in
 //                  it, and a list of row tiles (expert, first place, rows) for the products
-//   moe_gate_up    for every tile: y = act(A W_gate[e]^T, A W_up[e]^T), rows gathered by the permutation
+//   moe_gate_up    for every tile: y = act(A W_gate[e]^T, A W_up[e]^T), rows gathered by the permutation; or, for
+//                  experts without a gate, y = act(A W_up[e]^T)
 //   moe_down       for every tile: o = y W_down[e]^T, 32-bit
-//   moe_combine    delta[t] = sum_k weight[t,k] * o[place(t,k)], in the order of k
+//   moe_combine    delta[t] = sum_k weight[t,k] * o[place(t,k)], in the order of k, on top of `base` where given
 //   gated_act      the activation alone, for a dense feed-forward whose product left [gate | up]
 //
 // Activations (g = gate, u = up):
 //   0 silu:   g / (1 + exp(-g)) * u
 //   1 relu:   max(g, 0) * u
 //   2 clamped sigmoid gate: g' = min(g, limit), u' = clamp(u, -limit, limit); g' * sigmoid(alpha g') * (u' + shift)
+//   3 the tanh form of GELU on g, times u
+//   4 relu2:  max(g, 0)^2 * u
+// Without a gate the same functions of the one sum, with nothing to multiply (all but 2).
 //
 // The products run on the CUDA cores with 32-bit accumulation (every output element one
 // thread's sum over k in ascending order), so a row's result does not depend on where the
@@ -28,9 +35,11 @@
 #define ACT_RELU 1
 #define ACT_CLAMPED 2
 #define ACT_GELU_TANH 3
+#define ACT_RELU2 4
 
 __device__ __forceinline__ float gated_activation(float g, float u, int act, float limit, float alpha, float shift) {
     if (act == ACT_RELU) return fmaxf(g, 0.f) * u;
+    if (act == ACT_RELU2) { const float r = fmaxf(g, 0.f); return r * r * u; }
     if (act == ACT_GELU_TANH)        // 0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))) u
         return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
     if (act == ACT_CLAMPED) {
@@ -63,7 +72,7 @@ __global__ void gated_act_kernel(const TI* __restrict__ in, TO* __restrict__ out
 AP_EXPORT int ap_gated_act(const void* in, int in_dtype, void* out, int out_dtype, int T, int I, int pairs, int act,
                            float limit, float alpha, float shift, const float* row_scale, const int* scale_index,
                            cudaStream_t stream) {
-    AP_REQUIRE(T >= 0 && I > 0 && act >= 0 && act <= 3, "gated_act: bad sizes T=%d I=%d or activation %d", T, I, act);
+    AP_REQUIRE(T >= 0 && I > 0 && act >= 0 && act <= ACT_RELU2, "gated_act: bad sizes T=%d I=%d or activation %d", T, I, act);
     if (T == 0) return AP_OK;
     long long blocks = ((long long)T * I + 255) / 256;
     if (blocks > 148 * 32) blocks = 148 * 32;
@@ -85,6 +94,7 @@ AP_EXPORT int ap_gated_act(const void* in, int in_dtype, void* out, int out_dtyp
 #define ROUTE_TOP_SOFTMAX 0           // the `top` largest z + bias; shares: their softmax
 #define ROUTE_SOFTMAX_ALL 1           // s = softmax(z) over all; the `top` largest s + bias; shares: their s / sum
 #define ROUTE_SIGMOID 2               // s = sigmoid(z), each output alone; the `top` largest s + bias; shares: their s as it is
+#define ROUTE_SOFTMAX_SCORES 3        // as ROUTE_SOFTMAX_ALL, but the shares are the chosen s as they are
 
 // One CTA per RPB rows: eight warps, or, for a CTA of one row, a warp per router output (at most 32: a step of
 // few rows is a chain of loads per warp, which more warps shorten).  With `rows` the warps first form the rows' router logits: E dot
@@ -100,7 +110,7 @@ template <typename TA, typename TW, int RPB>
 __global__ void __launch_bounds__(ROUTE_MAX_THREADS)
 moe_route_kernel(const float* __restrict__ logits, const TA* __restrict__ rows, const TW* __restrict__ router, int K,
                  const float* __restrict__ bias, int* __restrict__ chosen, float* __restrict__ weight, int T, int E,
-                 int top, int mode) {
+                 int top, int mode, int groups, int keep, float share_scale) {
     __shared__ float z_all[RPB][32 * ROUTE_MAX_PER_LANE];
     ap_pdl_trigger();
     ap_pdl_wait();
@@ -156,7 +166,7 @@ moe_route_kernel(const float* __restrict__ logits, const TA* __restrict__ rows, 
     __syncthreads();
     if (warp >= nrows) return;
     const int t = t0 + warp;
-    const float* z_s = z_all[warp];
+    float* z_s = z_all[warp];
     float z[ROUTE_MAX_PER_LANE];
 #pragma unroll
     for (int i = 0; i < ROUTE_MAX_PER_LANE; ++i) {
@@ -166,7 +176,7 @@ moe_route_kernel(const float* __restrict__ logits, const TA* __restrict__ rows, 
     // ROUTE_SOFTMAX_ALL: scores s = softmax(z) over ALL experts; the choice goes by s + bias, the shares are
     // the chosen experts' s divided by their sum
     float sc[ROUTE_MAX_PER_LANE];
-    if (mode == ROUTE_SOFTMAX_ALL) {
+    if (mode == ROUTE_SOFTMAX_ALL || mode == ROUTE_SOFTMAX_SCORES) {
         float mx = -FLT_MAX;
 #pragma unroll
         for (int i = 0; i < ROUTE_MAX_PER_LANE; ++i) mx = fmaxf(mx, z[i]);
@@ -182,7 +192,8 @@ moe_route_kernel(const float* __restrict__ logits, const TA* __restrict__ rows, 
         for (int i = 0; i < ROUTE_MAX_PER_LANE; ++i) {
             const int e = lane + 32 * i;
             sc[i] /= sum;
-            z[i] = e < E ? sc[i] + (bias ? bias[e] : 0.f) : -FLT_MAX;
+            // without a bias the order of the scores is the order of the logits, which do not underflow
+            if (bias || mode == ROUTE_SOFTMAX_ALL) z[i] = e < E ? sc[i] + (bias ? bias[e] : 0.f) : -FLT_MAX;
         }
     } else if (mode == ROUTE_SIGMOID) {
 #pragma unroll
@@ -193,10 +204,50 @@ moe_route_kernel(const float* __restrict__ logits, const TA* __restrict__ rows, 
             z[i] = e < E ? (bias ? sc[i] + bias[e] : z[i]) : -FLT_MAX;
         }
     }
+    if (keep < groups) {
+        // what the choice goes by, in shared memory: a group's is its best expert's; a lane takes every 32nd group
+        const int each = E / groups;
+#pragma unroll
+        for (int i = 0; i < ROUTE_MAX_PER_LANE; ++i)
+            if (lane + 32 * i < E) z_s[lane + 32 * i] = z[i];
+        __syncwarp();
+        float gz[ROUTE_MAX_PER_LANE];
+#pragma unroll
+        for (int i = 0; i < ROUTE_MAX_PER_LANE; ++i) {
+            const int g = lane + 32 * i;
+            gz[i] = -FLT_MAX;
+            if (g < groups)
+                for (int e = g * each; e < (g + 1) * each; ++e) gz[i] = fmaxf(gz[i], z_s[e]);
+        }
+        unsigned open = 0;                                   // bit i: this lane's expert lane + 32 i may be chosen
+        for (int k = 0; k < keep; ++k) {
+            float v = -FLT_MAX;
+            int idx = 0x7fffffff;
+#pragma unroll
+            for (int i = 0; i < ROUTE_MAX_PER_LANE; ++i) {
+                const int g = lane + 32 * i;
+                if (g < groups && (gz[i] > v || (gz[i] == v && g < idx))) { v = gz[i]; idx = g; }
+            }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) {
+                const float ov = __shfl_xor_sync(0xffffffffu, v, o);
+                const int oi = __shfl_xor_sync(0xffffffffu, idx, o);
+                if (ov > v || (ov == v && oi < idx)) { v = ov; idx = oi; }
+            }
+#pragma unroll
+            for (int i = 0; i < ROUTE_MAX_PER_LANE; ++i) {
+                if (lane + 32 * i == idx) gz[i] = -INFINITY; // taken
+                if ((lane + 32 * i) / each == idx) open |= 1u << i;
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < ROUTE_MAX_PER_LANE; ++i)
+            if (!((open >> i) & 1u)) z[i] = -INFINITY;
+    }
     float best[ROUTE_MAX_TOP];
     int who[ROUTE_MAX_TOP];
     for (int k = 0; k < top; ++k) {
-        float v = -FLT_MAX;
+        float v = -INFINITY;
         int idx = 0x7fffffff;
 #pragma unroll
         for (int i = 0; i < ROUTE_MAX_PER_LANE; ++i) {
@@ -209,6 +260,7 @@ moe_route_kernel(const float* __restrict__ logits, const TA* __restrict__ rows, 
             const int oi = __shfl_xor_sync(0xffffffffu, idx, o);
             if (ov > v || (ov == v && oi < idx)) { v = ov; idx = oi; }
         }
+        if (idx >= E) idx = k;                               // (logits that are no numbers: some expert, never beyond the last)
         if (mode != ROUTE_TOP_SOFTMAX) {
             // the chosen expert's score without the bias: its owner's lane has it
             float own = 0.f;
@@ -221,26 +273,26 @@ moe_route_kernel(const float* __restrict__ logits, const TA* __restrict__ rows, 
         who[k] = idx;
 #pragma unroll
         for (int i = 0; i < ROUTE_MAX_PER_LANE; ++i)
-            if (lane + 32 * i == idx) z[i] = -FLT_MAX;        // taken
+            if (lane + 32 * i == idx) z[i] = -INFINITY;       // taken
     }
-    if (lane == 0 && mode == ROUTE_SIGMOID) {
+    if (lane == 0 && (mode == ROUTE_SIGMOID || mode == ROUTE_SOFTMAX_SCORES)) {
         for (int k = 0; k < top; ++k) {
             chosen[(size_t)t * top + k] = who[k];
-            weight[(size_t)t * top + k] = best[k];
+            weight[(size_t)t * top + k] = best[k] * share_scale;
         }
     } else if (lane == 0 && mode == ROUTE_SOFTMAX_ALL) {
         float sum = 0.f;
         for (int k = 0; k < top; ++k) sum += best[k];
         for (int k = 0; k < top; ++k) {
             chosen[(size_t)t * top + k] = who[k];
-            weight[(size_t)t * top + k] = best[k] / (sum + 1e-20f);
+            weight[(size_t)t * top + k] = best[k] / (sum + 1e-20f) * share_scale;
         }
     } else if (lane == 0) {
         float sum = 0.f;
         for (int k = 0; k < top; ++k) sum += expf(best[k] - best[0]);      // best[0] is the largest
         for (int k = 0; k < top; ++k) {
             chosen[(size_t)t * top + k] = who[k];
-            weight[(size_t)t * top + k] = expf(best[k] - best[0]) / sum;
+            weight[(size_t)t * top + k] = expf(best[k] - best[0]) / sum * share_scale;
         }
     }
 }
@@ -252,15 +304,17 @@ AP_EXPORT int ap_moe_route(const float* logits, const float* bias, int* chosen, 
     if (T == 0) return AP_OK;
     AP_CHECK_PDL_LAUNCH("moe_route", ap_launch_pdl(moe_route_kernel<float, float, 1>, dim3((unsigned)T), dim3(ROUTE_THREADS),
                                                    0, stream, logits, (const float*)nullptr, (const float*)nullptr, 0, bias,
-                                                   chosen, weight, T, E, top, ROUTE_TOP_SOFTMAX));
+                                                   chosen, weight, T, E, top, ROUTE_TOP_SOFTMAX, 1, 1, 1.0f));
     return AP_OK;
 }
 
 // the same from the rows themselves: rows [T, K], router [E, K]
 AP_EXPORT int ap_moe_route_rows(const void* rows, int rows_dtype, const void* router, int router_dtype, int K,
-                                const float* bias, int* chosen, float* weight, int T, int E, int top, int mode,
-                                cudaStream_t stream) {
-    AP_REQUIRE(mode == ROUTE_TOP_SOFTMAX || mode == ROUTE_SOFTMAX_ALL || mode == ROUTE_SIGMOID, "moe_route: unknown mode %d", mode);
+                                const float* bias, int* chosen, float* weight, int T, int E, int top, int mode, int groups,
+                                int keep, float share_scale, cudaStream_t stream) {
+    AP_REQUIRE(mode >= ROUTE_TOP_SOFTMAX && mode <= ROUTE_SOFTMAX_SCORES, "moe_route: unknown mode %d", mode);
+    AP_REQUIRE(groups > 0 && E % groups == 0 && keep > 0 && keep <= groups && top <= E / groups * keep,
+               "moe_route: %d experts in %d groups, %d of them kept, %d chosen", E, groups, keep, top);
     AP_REQUIRE(T >= 0 && K > 0 && E > 0 && E <= 32 * ROUTE_MAX_PER_LANE && top > 0 && top <= E && top <= ROUTE_MAX_TOP,
                "moe_route: %d experts (at most %d), %d chosen (at most %d)", E, 32 * ROUTE_MAX_PER_LANE, top, ROUTE_MAX_TOP);
     if (T == 0) return AP_OK;
@@ -271,7 +325,7 @@ AP_EXPORT int ap_moe_route_rows(const void* rows, int rows_dtype, const void* ro
     AP_CHECK_PDL_LAUNCH("moe_route", ap_launch_pdl(moe_route_kernel<TA, TW, R>, dim3((unsigned)((T + R - 1) / R)),   \
                                                    dim3(R == 1 ? threads1 : ROUTE_THREADS), 0, stream, (const float*)nullptr,           \
                                                    (const TA*)rows, (const TW*)router, K, bias, chosen, weight, T, E, \
-                                                   top, mode))
+                                                   top, mode, groups, keep, share_scale))
 #define LAUNCH(TA, TW) do { if (four) LAUNCH_R(TA, TW, 4); else LAUNCH_R(TA, TW, 1); } while (0)
     if (rows_dtype == AP_F32 && router_dtype == AP_F32) LAUNCH(float, float);
     else if (rows_dtype == AP_BF16 && router_dtype == AP_BF16) LAUNCH(bf16, bf16);
@@ -340,10 +394,10 @@ AP_EXPORT int ap_moe_sort(const int* chosen, int* perm, int* place, int* tiles, 
 }
 
 // ---- the experts' products ---------------------------------------------------------------
-// GATED: the weight of expert e is [2 F, K] (gate rows, then up rows); out[p, f] = act(gate, up).
-// else : the weight is [N, K]; out[p, n] 32-bit.
-// A rows: GATED gathers a[perm[p] / top]; else a[p].
-template <typename TA, typename TW, typename TO, bool GATED>
+// FIRST: the experts' first product.  A rows are gathered, a[perm[p] / top].  GATED: the weight of expert e is [2 F, K]
+//         (gate rows, then up rows), out[p, f] = act(gate, up); else [F, K], out[p, f] = act(up).
+// else : the weight is [N, K]; A row a[p]; out[p, n] 32-bit.
+template <typename TA, typename TW, typename TO, bool FIRST, bool GATED>
 __global__ void __launch_bounds__(256)
 moe_gemm_kernel(const TA* __restrict__ A, long long lda, const TW* __restrict__ W, long long w_expert_stride,
                 TO* __restrict__ C, long long ldc, const int* __restrict__ perm, int top, const int3* __restrict__ tiles,
@@ -361,7 +415,7 @@ moe_gemm_kernel(const TA* __restrict__ A, long long lda, const TW* __restrict__ 
     const int tx = tid & 15, ty = tid >> 4;
     const int n0 = blockIdx.x * MOE_BN;
     const TW* We = W + (size_t)e * w_expert_stride;
-    if (tid < MOE_BM) src_row[tid] = tid < rows ? (GATED ? perm[p0 + tid] / top : p0 + tid) : -1;
+    if (tid < MOE_BM) src_row[tid] = tid < rows ? (FIRST ? perm[p0 + tid] / top : p0 + tid) : -1;
     __syncthreads();
     float acc[4][4], acc2[GATED ? 4 : 1][4];
 #pragma unroll
@@ -413,10 +467,11 @@ moe_gemm_kernel(const TA* __restrict__ A, long long lda, const TW* __restrict__ 
             const int n = n0 + tx * 4 + j;
             if (n >= N) continue;
             float v = acc[i][j];
-            if constexpr (GATED) {
+            if constexpr (FIRST) {
                 // a scale of the pair's INPUT row multiplies both sums
                 const float sc = pair_scale ? pair_scale[perm[p0 + r]] : 1.0f;
-                v = gated_activation(acc[i][j] * sc, acc2[i][j] * sc, act, limit, alpha, shift);
+                if constexpr (GATED) v = gated_activation(acc[i][j] * sc, acc2[i][j] * sc, act, limit, alpha, shift);
+                else v = gated_activation(v * sc, 1.0f, act, 0.f, 0.f, 0.f);
             }
             C[(size_t)(p0 + r) * ldc + n] = ap_from_float<TO>(v);
         }
@@ -453,7 +508,7 @@ __device__ __forceinline__ float moe_rows_sum8(const float* acc, int lane) {
     return a1;
 }
 
-template <bool GATED, typename TO>
+template <bool FIRST, bool GATED, typename TO>
 __global__ void __launch_bounds__(256)
 moe_rows_kernel(const bf16* __restrict__ A, long long lda, const bf16* __restrict__ W, long long w_expert_stride,
                 TO* __restrict__ C, long long ldc, const int* __restrict__ perm, int top, const int3* __restrict__ tiles,
@@ -475,7 +530,7 @@ moe_rows_kernel(const bf16* __restrict__ A, long long lda, const bf16* __restric
             const int r = i / K8, c = i - r * K8;
             uint4 v = make_uint4(0, 0, 0, 0);
             if (r < R) {
-                const int src = GATED ? perm[p0 + r0 + r] / top : p0 + r0 + r;
+                const int src = FIRST ? perm[p0 + r0 + r] / top : p0 + r0 + r;
                 v = *reinterpret_cast<const uint4*>(A + (size_t)src * lda + c * 8);
             }
             *reinterpret_cast<uint4*>(a_s + (size_t)r * K + c * 8) = v;
@@ -529,9 +584,10 @@ moe_rows_kernel(const bf16* __restrict__ A, long long lda, const bf16* __restric
             float v = moe_rows_sum8(acc, lane), v2 = 0.f;
             if constexpr (GATED) v2 = moe_rows_sum8(acc2, lane);
             if ((lane & 3) == 0 && out_row < R) {
-                if constexpr (GATED) {
+                if constexpr (FIRST) {
                     const float sc = pair_scale ? pair_scale[perm[p0 + r0 + out_row]] : 1.0f;
-                    v = gated_activation(v * sc, v2 * sc, act, limit, alpha, shift);
+                    if constexpr (GATED) v = gated_activation(v * sc, v2 * sc, act, limit, alpha, shift);
+                    else v = gated_activation(v * sc, 1.0f, act, 0.f, 0.f, 0.f);
                 }
                 C[(size_t)(p0 + r0 + out_row) * ldc + n] = ap_from_float<TO>(v);
             }
@@ -545,30 +601,33 @@ static bool moe_few_rows(int pairs, int E, int K, const void* a, const void* w) 
            ((((uintptr_t)a) | ((uintptr_t)w)) & 15) == 0;
 }
 
-// a: [T, K]; w_gate_up: [E, 2 F, K]; y: [pairs, F] in the activation type
+// a: [T, K]; w_gate_up: [E, 2 F, K], or (not `gated`) [E, F, K]; y: [pairs, F] in the activation type
 AP_EXPORT int ap_moe_gate_up(const void* a, int a_dtype, const void* w, int w_dtype, void* y, int y_dtype,
-                             const int* perm, int top, const int* tiles, int pairs, int E, int F, int K, int act,
+                             const int* perm, int top, const int* tiles, int pairs, int E, int F, int K, int gated, int act,
                              float limit, float alpha, float shift, const float* pair_scale, cudaStream_t stream) {
-    AP_REQUIRE(pairs >= 0 && E > 0 && F > 0 && K > 0 && top > 0 && act >= 0 && act <= 3, "moe_gate_up: bad sizes");
+    AP_REQUIRE(pairs >= 0 && E > 0 && F > 0 && K > 0 && top > 0 && act >= 0 && act <= ACT_RELU2, "moe_gate_up: bad sizes");
+    AP_REQUIRE(gated || act != ACT_CLAMPED, "moe_gate_up: activation %d needs a gate", act);
     if (pairs == 0) return AP_OK;
     const int max_tiles = ap_moe_max_tiles(pairs, E);
     const dim3 grid((unsigned)((F + MOE_BN - 1) / MOE_BN), (unsigned)max_tiles);
     AP_REQUIRE(max_tiles <= 65535, "moe_gate_up: %d row tiles exceed the grid", max_tiles);
-#define LAUNCH(TA, TW, TO)                                                                                           \
-    AP_CHECK_PDL_LAUNCH("moe_gate_up", ap_launch_pdl(moe_gemm_kernel<TA, TW, TO, true>, grid, dim3(256), 0, stream,  \
-                                                     (const TA*)a, (long long)K, (const TW*)w, (long long)2 * F * K, \
+    const long long expert_stride = (long long)(gated ? 2 : 1) * F * K;
+#define LAUNCH(TA, TW, TO) do { if (gated) LAUNCH_G(TA, TW, TO, true); else LAUNCH_G(TA, TW, TO, false); } while (0)
+#define LAUNCH_G(TA, TW, TO, G)                                                                                      \
+    AP_CHECK_PDL_LAUNCH("moe_gate_up", ap_launch_pdl(moe_gemm_kernel<TA, TW, TO, true, G>, grid, dim3(256), 0, stream,  \
+                                                     (const TA*)a, (long long)K, (const TW*)w, expert_stride, \
                                                      (TO*)y, (long long)F, perm, top, (const int3*)tiles, max_tiles, F, K, \
                                                      act, limit, alpha, shift, pair_scale))
     if (a_dtype == AP_BF16 && w_dtype == AP_BF16 && y_dtype == AP_BF16 && moe_few_rows(pairs, E, K, a, w)) {
         const dim3 rgrid((unsigned)((F + ROWS_COLS - 1) / ROWS_COLS), (unsigned)max_tiles);
         const size_t smem = (size_t)ROWS_MAX * K * sizeof(bf16);
-        auto kern = moe_rows_kernel<true, bf16>;
+        auto kern = gated ? moe_rows_kernel<true, true, bf16> : moe_rows_kernel<true, false, bf16>;
         if (smem > 48 * 1024) {
             cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
             AP_REQUIRE(e == cudaSuccess, "moe_gate_up: cannot reserve %zu bytes of shared memory", smem);
         }
         AP_CHECK_PDL_LAUNCH("moe_gate_up", ap_launch_pdl(kern, rgrid, dim3(256), smem, stream, (const bf16*)a, (long long)K,
-                                                         (const bf16*)w, (long long)2 * F * K, (bf16*)y, (long long)F, perm,
+                                                         (const bf16*)w, expert_stride, (bf16*)y, (long long)F, perm,
                                                          top, (const int3*)tiles, max_tiles, F, K, act, limit, alpha, shift, pair_scale));
         return AP_OK;
     }
@@ -577,6 +636,7 @@ AP_EXPORT int ap_moe_gate_up(const void* a, int a_dtype, const void* w, int w_dt
     else if (a_dtype == AP_BF16 && w_dtype == AP_F32 && y_dtype == AP_BF16) LAUNCH(bf16, float, bf16);
     else AP_REQUIRE(false, "moe_gate_up: unsupported dtypes a=%d w=%d y=%d", a_dtype, w_dtype, y_dtype);
 #undef LAUNCH
+#undef LAUNCH_G
     return AP_OK;
 }
 
@@ -589,14 +649,14 @@ AP_EXPORT int ap_moe_down(const void* y, int y_dtype, const void* w, int w_dtype
     const dim3 grid((unsigned)((H + MOE_BN - 1) / MOE_BN), (unsigned)max_tiles);
     AP_REQUIRE(max_tiles <= 65535, "moe_down: %d row tiles exceed the grid", max_tiles);
 #define LAUNCH(TA, TW)                                                                                               \
-    AP_CHECK_PDL_LAUNCH("moe_down", ap_launch_pdl(moe_gemm_kernel<TA, TW, float, false>, grid, dim3(256), 0, stream, \
+    AP_CHECK_PDL_LAUNCH("moe_down", ap_launch_pdl(moe_gemm_kernel<TA, TW, float, false, false>, grid, dim3(256), 0, stream, \
                                                   (const TA*)y, (long long)F, (const TW*)w, (long long)H * F, o,     \
                                                   (long long)H, (const int*)nullptr, 1, (const int3*)tiles, max_tiles, H, \
                                                   F, 0, 0.f, 0.f, 0.f, (const float*)nullptr))
     if (y_dtype == AP_BF16 && w_dtype == AP_BF16 && moe_few_rows(pairs, E, F, y, w)) {
         const dim3 rgrid((unsigned)((H + ROWS_COLS - 1) / ROWS_COLS), (unsigned)max_tiles);
         const size_t smem = (size_t)ROWS_MAX * F * sizeof(bf16);
-        auto kern = moe_rows_kernel<false, float>;
+        auto kern = moe_rows_kernel<false, false, float>;
         if (smem > 48 * 1024) {
             cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
             AP_REQUIRE(e == cudaSuccess, "moe_down: cannot reserve %zu bytes of shared memory", smem);
@@ -643,13 +703,14 @@ AP_EXPORT int ap_moe_gather(const void* a, void* out, const int* perm, int top, 
 template <typename TA>
 __global__ void moe_combine_kernel(const float* __restrict__ o, const int* __restrict__ place,
                                    const float* __restrict__ weight, float* __restrict__ delta, int T, int H, int top,
-                                   const int* __restrict__ chosen, int real, const TA* __restrict__ rows) {
+                                   const int* __restrict__ chosen, int real, const TA* __restrict__ rows,
+                                   const float* __restrict__ base) {
     ap_pdl_trigger();
     ap_pdl_wait();
     const size_t n = (size_t)T * H;
     for (size_t e = blockIdx.x * (size_t)blockDim.x + threadIdx.x; e < n; e += (size_t)gridDim.x * blockDim.x) {
         const size_t t = e / H, c = e - t * H;
-        float v = 0.f;
+        float v = base ? base[e] : 0.f;
         for (int k = 0; k < top; ++k) {
             const bool identity = chosen != nullptr && chosen[t * top + k] >= real;
             v = fmaf(weight ? weight[t * top + k] : 1.0f, identity ? ap_to_float(rows[e]) : o[(size_t)place[t * top + k] * H + c], v);
@@ -659,7 +720,8 @@ __global__ void moe_combine_kernel(const float* __restrict__ o, const int* __res
 }
 
 AP_EXPORT int ap_moe_combine(const float* o, const int* place, const float* weight, float* delta, int T, int H, int top,
-                             const int* chosen, int real, const void* rows, int rows_dtype, cudaStream_t stream) {
+                             const int* chosen, int real, const void* rows, int rows_dtype, const float* base,
+                             cudaStream_t stream) {
     AP_REQUIRE(T >= 0 && H > 0 && top > 0, "moe_combine: bad sizes");
     AP_REQUIRE(chosen == nullptr || rows != nullptr, "moe_combine: identity experts need the rows' input");
     if (T == 0) return AP_OK;
@@ -668,10 +730,10 @@ AP_EXPORT int ap_moe_combine(const float* o, const int* place, const float* weig
     if (chosen != nullptr && rows_dtype == AP_BF16)
         AP_CHECK_PDL_LAUNCH("moe_combine", ap_launch_pdl(moe_combine_kernel<bf16>, dim3((unsigned)blocks), dim3(256), 0,
                                                          stream, o, place, weight, delta, T, H, top, chosen, real,
-                                                         (const bf16*)rows));
+                                                         (const bf16*)rows, base));
     else
         AP_CHECK_PDL_LAUNCH("moe_combine", ap_launch_pdl(moe_combine_kernel<float>, dim3((unsigned)blocks), dim3(256), 0,
                                                          stream, o, place, weight, delta, T, H, top, chosen, real,
-                                                         (const float*)rows));
+                                                         (const float*)rows, base));
     return AP_OK;
 }

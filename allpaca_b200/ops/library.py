@@ -81,19 +81,20 @@ _CORE_SIGNATURES = {
     # int ap_gated_act(in, in_dtype, out, out_dtype, T, I, pairs, act, limit, alpha, shift, row_scale, scale_index, stream)
     "ap_gated_act": [_P, _I, _P, _I, _I, _I, _I, _I, _F, _F, _F, _P, _P, _P],
     "ap_moe_route": [_P, _P, _P, _P, _I, _I, _I, _P],
-    # int ap_moe_route_rows(rows, rows_dtype, router, router_dtype, K, bias, chosen, weight, T, E, top, mode, stream)
-    "ap_moe_route_rows": [_P, _I, _P, _I, _I, _P, _P, _P, _I, _I, _I, _I, _P],
+    # int ap_moe_route_rows(rows, rows_dtype, router, router_dtype, K, bias, chosen, weight, T, E, top, mode, groups,
+    #                       keep, share_scale, stream)
+    "ap_moe_route_rows": [_P, _I, _P, _I, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _P],
     "ap_moe_max_tiles": [_I, _I],
     # int ap_moe_sort(chosen, perm, place, tiles, offsets, pairs, E, real, stream)
     "ap_moe_sort": [_P, _P, _P, _P, _P, _I, _I, _I, _P],
     "ap_moe_gather": [_P, _P, _P, _I, _I, _I, _P],
-    # int ap_moe_gate_up(a, a_dtype, w, w_dtype, y, y_dtype, perm, top, tiles, pairs, E, F, K, act, limit, alpha,
-    #                    shift, pair_scale, stream)
-    "ap_moe_gate_up": [_P, _I, _P, _I, _P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _F, _F, _F, _P, _P],
+    # int ap_moe_gate_up(a, a_dtype, w, w_dtype, y, y_dtype, perm, top, tiles, pairs, E, F, K, gated, act, limit,
+    #                    alpha, shift, pair_scale, stream)
+    "ap_moe_gate_up": [_P, _I, _P, _I, _P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _F, _F, _F, _P, _P],
     # int ap_moe_down(y, y_dtype, w, w_dtype, o, tiles, pairs, E, H, F, stream)
     "ap_moe_down": [_P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _P],
-    # int ap_moe_combine(o, place, weight, delta, T, H, top, chosen, real, rows, rows_dtype, stream)
-    "ap_moe_combine": [_P, _P, _P, _P, _I, _I, _I, _P, _I, _P, _I, _P],
+    # int ap_moe_combine(o, place, weight, delta, T, H, top, chosen, real, rows, rows_dtype, base, stream)
+    "ap_moe_combine": [_P, _P, _P, _P, _I, _I, _I, _P, _I, _P, _I, _P, _P],
     # int ap_add_dyt(x, delta, S, delta_stride, w, b, alpha, out, out_dtype, rows, R, H, stream)
     "ap_add_dyt": [_P, _P, _I, _L, _P, _P, _F, _P, _I, _P, _I, _I, _P],
     # int ap_dyt_shift(x, w, b, alpha, shift, state, state_stride, seq_start, positions, token_seq, state_slots,
@@ -103,12 +104,17 @@ _CORE_SIGNATURES = {
     "ap_stream_mix": [_P, _P, _I, _L, _P, _L, _I, _P, _L, _P],
     # int ap_linear_scan(q, ld_q, k, ld_k, v, ld_v, decay_channel, ld_dc, decay_head, ld_dh, decay_const, dt_bias, beta,
     #                    ld_beta, cos_sin, rot_dims, state, state_stride, seq_start, positions, state_slots, y, ld_y,
-    #                    T, nseq, heads, qk_heads, D, V, decay_mode, qk_mode, tau, unit_eps, out_scale, scratch, stream)
+    #                    T, nseq, heads, qk_heads, D, V, decay_mode, qk_mode, delta, unit_column, tau, unit_eps,
+    #                    out_scale, scratch, stream)
     "ap_linear_scan": [_P, _L, _P, _L, _P, _L, _P, _L, _P, _L, _P, _P, _P, _L, _P, _I, _P, _L, _P, _P, _P, _P, _L,
-                       _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _P, _P],
+                       _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _P, _P],
+    # int ap_exp_gates(raw_i, raw_f, ld, bias_i, bias_f, cap, state, state_stride, seq_start, positions, state_slots,
+    #                  floor, T, nseq, heads, stream)
+    "ap_exp_gates": [_P, _P, _L, _P, _P, _F, _P, _L, _P, _P, _P, _P, _I, _I, _I, _P],
     "ap_linear_scan_block": [_I, _I, _I, _I, _I, _I],
-    # int ap_head_norm_gate(y, ld_y, gate, ld_g, w, eps, out_scale, act, out, out_dtype, T, heads, V, stream)
-    "ap_head_norm_gate": [_P, _L, _P, _L, _P, _F, _F, _I, _P, _I, _I, _I, _I, _P],
+    # int ap_head_norm_gate(y, ld_y, head_stride, floor, floor_eps, gate, ld_g, w, own_weights, eps, out_scale, act, out,
+    #                       out_dtype, T, heads, V, stream)
+    "ap_head_norm_gate": [_P, _L, _I, _P, _F, _P, _L, _P, _I, _F, _F, _I, _P, _I, _I, _I, _I, _P],
     # int ap_stream_norm(x, rows, R, delta, S, slice_stride, slice_bias, slice_w, slice_eps, slice_scale, out_w, mix,
     #                    in_w, w, eps, update, out, out_dtype, streams, H, stream)
     "ap_stream_norm": [_P, _P, _I, _P, _I, _L, _P, _P, _F, _F, _P, _P, _P, _P, _F, _I, _P, _I, _I, _I, _P],

@@ -68,7 +68,8 @@ def qk_norm_store(qkv: torch.Tensor, q_out: torch.Tensor, cache_layer: Optional[
     (32-bit ``[D]``, shared by the heads; None: no weight), queries multiplied by
     ``1 + temp_coef * ln(floor((pos + 1) / temp_every) + 1)`` (``temp_every`` 0: no temperature) into
     ``q_out [T, nh*D]``, keys and values into the pages ``cache_layer [pages, nkv, P, D + VD]``
-    (None: not stored).  ``bias`` (32-bit, one number per column of Q, K and V) is added to the sums as they are
+    (None: only the queries are made ready, and ``qkv`` and ``bias`` need not hold more than theirs).  ``bias`` (32-bit,
+    one number per column of Q, K and V) is added to the sums as they are
     read; ``cos_sin [T, r/2, 2]`` turns the first ``r`` coordinates of every normed query and key head, coordinate
     ``i`` with ``i + r/2`` (``pairing`` 0) or ``2i`` with ``2i + 1`` (1); values are multiplied by ``value_scale`` on their way into the page."""
     if qkv.dim() != 2 or not qkv.is_cuda or qkv.stride(1) != 1:
@@ -80,8 +81,9 @@ def qk_norm_store(qkv: torch.Tensor, q_out: torch.Tensor, cache_layer: Optional[
             _check(w, n, torch.float32, 1)
             if w.shape[0] != key_dim:
                 raise KernelError(f"qk_norm_store: {n} must have one entry per coordinate of a head")
-    if qkv.shape[1] < (num_heads + num_kv_heads) * key_dim + num_kv_heads * value_dim \
-            or q_out.shape[0] < T or q_out.shape[1] != num_heads * key_dim:
+    stored = num_kv_heads if cache_layer is not None else 0
+    columns = (num_heads + stored) * key_dim + stored * value_dim
+    if qkv.shape[1] < columns or q_out.shape[0] < T or q_out.shape[1] != num_heads * key_dim:
         raise KernelError(f"qk_norm_store: shapes disagree: qkv {tuple(qkv.shape)}, q_out {tuple(q_out.shape)}")
     _check(positions, "positions", torch.int32, 1)
     rot_dims = 0
@@ -92,7 +94,7 @@ def qk_norm_store(qkv: torch.Tensor, q_out: torch.Tensor, cache_layer: Optional[
             raise KernelError(f"qk_norm_store: cos_sin {tuple(cos_sin.shape)} is not [T, r/2, 2] with r <= {key_dim}")
     if bias is not None:
         _check(bias, "bias", torch.float32, 1)
-        if bias.shape[0] != (num_heads + num_kv_heads) * key_dim + num_kv_heads * value_dim:
+        if bias.shape[0] < columns:
             raise KernelError("qk_norm_store: the bias must have one entry per column of Q, K and V")
     P, page_stride, cptr, tsptr, btptr, maxb = 1, 0, 0, 0, 0, 0
     if cache_layer is not None:

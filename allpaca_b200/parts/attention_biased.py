@@ -26,8 +26,13 @@
   ``q.conv``, ``k.conv``, ``v.conv`` ``[channels, n]``, the last column on the row itself, zeros before the sequence's
   start, no activation), after the bias and before norm and rotation; the last ``n - 1`` biased projections are
   fixed-size state of the request, 32-bit;
-* ``sink``: the softmax's denominator also holds ``exp(sink[h])``, one learned number per query head (tensor
-  ``sink``) to which neither key nor value belongs;
+* ``sink``: the softmax's denominator also holds ``exp(sink[h])``, to which neither key nor value belongs: True: one
+  learned number per query head (tensor ``sink``); a number: that one for every head (0: the denominator is
+  ``1 + sum``); no tensor;
+* ``shares_kv``: the layer has no K and V and reads the keys and values another layer's run keeps (the model's order
+  names that run as this run's ``cache_from``), with its own queries, window and everything else; ``cache_window``: how
+  far back the pages must stay readable, which is the largest window among this layer and the layers that read its keys
+  and values (None where one of them has no window; left out: this layer's own window);
 * ``output_scale``: the mixer's result times a constant (carried by the values on their way into the pages, so
   that it costs nothing).
 
@@ -52,7 +57,7 @@ class DistanceBiasedAttention(Mixer):
     """Parameters: ``hidden_size``, ``num_heads``, ``num_kv_heads``, ``head_dim``, ``value_dim``
     (None: ``head_dim``), ``scale``, ``window``, ``keep_first``, ``qk_norm_eps``, ``qk_norm_weights``,
     ``q_temp``, ``distance_bias``, ``slope_exponent``, ``output_gate``, ``rope``, ``softcap``, ``qkv_bias``,
-    ``o_bias``, ``conv_taps``, ``sink``, ``output_scale``; tensors ``q``, ``k``, ``v``, ``o``
+    ``o_bias``, ``conv_taps``, ``sink``, ``shares_kv``, ``cache_window``, ``output_scale``; tensors ``q``, ``k``, ``v``, ``o``
     (``[out, in]``) and, by the parameters, ``r1``, ``r2``, ``sink`` (``[num_heads]``), ``q.norm``, ``k.norm``
     (``[head_dim]``), ``g`` (``[num_heads, hidden]``), ``q.b``, ``k.b``, ``v.b``, ``o.b``, ``q.conv``, ``k.conv``,
     ``v.conv``."""
@@ -92,7 +97,14 @@ class DistanceBiasedAttention(Mixer):
         if self.qk_norm_weights and self.qk_norm_eps is None:
             raise PartError("qk_norm_weights needs qk_norm_eps")
         self.output_gate = bool(p.get("output_gate", False))
-        self.q_size, self.k_size, self.v_size = self.nh * self.hd, self.nkv * self.hd, self.nkv * self.vd
+        self.shares_kv = bool(p.get("shares_kv", False))
+        if self.shares_kv and (p.get("conv_taps") or self.keep_first):
+            raise PartError("a layer that reads another's keys and values has no convolution and keeps no first tokens")
+        self.cache_window = p["cache_window"] if "cache_window" in p else self.window
+        if self.cache_window is not None and (self.window is None or self.cache_window < self.window):
+            raise PartError("an attention layer's pages must stay readable as far back as its window reaches")
+        self.q_size = self.nh * self.hd
+        self.k_size, self.v_size = (0, 0) if self.shares_kv else (self.nkv * self.hd, self.nkv * self.vd)
         self.g_size = self.nh if self.output_gate else 0
         self.qkv = Linear(env, self.q_size + self.k_size + self.v_size + self.g_size, self.hidden)
         self.o = Linear(env, self.hidden, self.nh * self.vd)
@@ -107,7 +119,9 @@ class DistanceBiasedAttention(Mixer):
         self.taps = int(p.get("conv_taps") or 0)
         self.conv_channels = self.q_size + self.k_size + self.v_size
         self.conv_w = self.sink = None
-        self.has_sink = bool(p.get("sink", False))
+        sink = p.get("sink", False)
+        self.has_sink = sink is True                          # learned numbers
+        self.fixed_sink = float(sink) if not isinstance(sink, bool) and sink is not None else None
         self.output_scale = float(p.get("output_scale", 1.0))
 
     def state_bytes(self) -> int:
@@ -119,19 +133,22 @@ class DistanceBiasedAttention(Mixer):
             yield from self.position.parts()
 
     def weights(self) -> Dict[str, WeightSpec]:
-        w = {"q": WeightSpec((self.q_size, self.hidden)), "k": WeightSpec((self.k_size, self.hidden)),
-             "v": WeightSpec((self.v_size, self.hidden)), "o": WeightSpec((self.hidden, self.nh * self.vd))}
+        w = {"q": WeightSpec((self.q_size, self.hidden)), "o": WeightSpec((self.hidden, self.nh * self.vd))}
+        if not self.shares_kv:
+            w.update({"k": WeightSpec((self.k_size, self.hidden)), "v": WeightSpec((self.v_size, self.hidden))})
         if self.distance_bias:
             w["r1"] = WeightSpec((self.nh,), "positive")
             w["r2"] = WeightSpec((self.nh,), "positive")
         if self.qk_norm_weights:
             w["q.norm"] = WeightSpec((self.hd,), "norm")
-            w["k.norm"] = WeightSpec((self.hd,), "norm")
+            if not self.shares_kv:
+                w["k.norm"] = WeightSpec((self.hd,), "norm")
         if self.output_gate:
             w["g"] = WeightSpec((self.nh, self.hidden))
         if self.has_qkv_bias:
-            w.update({"q.b": WeightSpec((self.q_size,), "bias"), "k.b": WeightSpec((self.k_size,), "bias"),
-                      "v.b": WeightSpec((self.v_size,), "bias")})
+            w["q.b"] = WeightSpec((self.q_size,), "bias")
+            if not self.shares_kv:
+                w.update({"k.b": WeightSpec((self.k_size,), "bias"), "v.b": WeightSpec((self.v_size,), "bias")})
         if self.has_o_bias:
             w["o.b"] = WeightSpec((self.hidden,), "bias")
         if self.taps > 0:
@@ -143,7 +160,8 @@ class DistanceBiasedAttention(Mixer):
         return w
 
     def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
-        stacked = [tensors["q"], tensors["k"], tensors["v"]] + ([tensors["g"]] if self.output_gate else [])
+        own = ("q",) if self.shares_kv else ("q", "k", "v")
+        stacked = [tensors[n] for n in own] + ([tensors["g"]] if self.output_gate else [])
         self.qkv.load(torch.cat(stacked, dim=0))
         self.o.load(tensors["o"])
         if self.distance_bias:
@@ -155,19 +173,21 @@ class DistanceBiasedAttention(Mixer):
             self.r1 = torch.pow(torch.tensor(2.0, dtype=torch.float64), -self.slope_exponent * h / self.nh) \
                 .to(torch.float32).to(self.env.device)
         if self.has_qkv_bias:
-            self.qkv_bias = torch.cat([tensors["q.b"], tensors["k.b"], tensors["v.b"]]).float().contiguous()
+            self.qkv_bias = torch.cat([tensors[n + ".b"] for n in own]).float().contiguous()
         if self.has_o_bias:
             self.output_bias = (tensors["o.b"].float() * self.output_scale).contiguous()
         if self.taps > 0:
             self.conv_w = torch.cat([tensors["q.conv"], tensors["k.conv"], tensors["v.conv"]], dim=0).float().contiguous()
         if self.has_sink:
             self.sink = tensors["sink"].float().contiguous()
+        elif self.fixed_sink is not None:
+            self.sink = torch.full((self.nh,), self.fixed_sink, dtype=torch.float32, device=self.env.device)
         if self.qk_norm_weights:
             self.q_weight = tensors["q.norm"].float().contiguous()
-            self.k_weight = tensors["k.norm"].float().contiguous()
+            self.k_weight = tensors["k.norm"].float().contiguous() if not self.shares_kv else None
 
     def cache_need(self) -> Optional[CacheNeed]:
-        return CacheNeed(outer=(self.nkv,), inner=(self.hd + self.vd,), window=self.window,
+        return CacheNeed(outer=(self.nkv,), inner=(self.hd + self.vd,), window=self.cache_window,
                          keep_first=self.keep_first)
 
     def forward(self, h: torch.Tensor, step, cache: LayerCache, into=None, add_bias: bool = True) -> torch.Tensor:
@@ -175,6 +195,8 @@ class DistanceBiasedAttention(Mixer):
         that runs beside another one; ``add_bias`` False: the caller adds ``output_bias`` itself."""
         T = h.shape[0]
         ws = self.env.workspace
+        if cache.writes == self.shares_kv:
+            raise PartError("an attention layer writes pages exactly when it has keys and values of its own")
         proj = qkv = self.qkv.forward(h, "battn.qkv", "float32")
         bias = self.qkv_bias
         if self.taps > 0:

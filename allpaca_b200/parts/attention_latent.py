@@ -9,8 +9,11 @@ query/key dimensions, values of ``value_dim`` and a latent of ``kv_rank``:
   the latent ``c``; the last ``rot_dim``, not normed, are one rotated key part all heads share;
 * head ``a`` has the unrotated key ``W_uk[a] c`` and the value ``W_uv[a] c``;
   ``score = (q_unrotated . k_unrotated + q_rotated . k_rotated) * scale``, causal, ordinary softmax;
-* the rotation (``rope``: ``dims``, ``theta``, ``scaling``, see :mod:`.rope`) acts on the first ``dims`` of
-  the ``rot_dim`` rotated dimensions of queries and of the shared key part, never on values;
+* the rotation (``rope``: ``dims``, ``theta``, ``scaling``, ``pairing``, see :mod:`.rope`) acts on the first ``dims`` of
+  the ``rot_dim`` rotated dimensions of queries and of the shared key part, never on values.  The kernels turn
+  coordinate ``i`` with ``i + dims/2``; for a ``pairing`` of neighbours (``"adjacent"``) the rows of the matrices that
+  form the rotated parts are reordered once, at load, so that the pairs lie that way: a score is a sum over the
+  coordinates, whose order does not matter to it;
 * ``output_gate``: head ``a`` of the result is multiplied by ``sigmoid(W_g h)_a`` before ``W_o``;
 * ``shares_latent``: the layer has no ``W_dkv`` and reads the latent and the rotated key part another
   layer's run keeps (the model's order names that run as this run's ``cache_from``), with its own
@@ -47,12 +50,13 @@ import torch
 from .. import ops
 from .base import BuildEnv, CacheNeed, LayerCache, Mixer, PartError, PartSpec, WeightSpec, build, register
 from .linear import Linear
+from .rope import PAIRING
 
 
 @register("mixer", "latent_attention")
 class LatentAttention(Mixer):
     """Parameters: ``hidden_size``, ``num_heads``, ``head_dim``, ``rot_dim``, ``value_dim``, ``kv_rank``,
-    ``q_rank`` (0: none), ``scale``, ``norm_eps``, ``rope`` (``{"dims", "theta", "scaling"}``), ``output_gate``,
+    ``q_rank`` (0: none), ``scale``, ``norm_eps``, ``rope`` (``{"dims", "theta", "scaling", "pairing"}``), ``output_gate``,
     ``shares_latent``, ``window`` (None), ``cache_window`` (the window), ``sink`` (False); tensors ``dq``,
     ``dq.norm``, ``uq`` (or ``q`` without a query latent), ``dkv``, ``dkv.norm`` (both absent with
     ``shares_latent``), ``uk``, ``uv``, ``g`` (with ``output_gate``), ``sink`` (with ``sink``), ``o``."""
@@ -83,6 +87,7 @@ class LatentAttention(Mixer):
         rope = p.get("rope")
         self.rope = None
         self.rot_dims = 0
+        self.rot_order = None         # where the rotated part's coordinates come from (None: as they are stored)
         if rope and self.rot > 0:
             self.rot_dims = int(rope["dims"])
             if self.rot_dims % 2 or not (0 < self.rot_dims <= self.rot):
@@ -90,6 +95,12 @@ class LatentAttention(Mixer):
             self.rope = build("position", PartSpec("rope", {
                 "head_dim": self.rot_dims, "theta": float(rope["theta"]), "scaling": rope.get("scaling"),
                 "pairing": "half"}), env)
+            pairing = rope.get("pairing", "half")
+            if pairing not in PAIRING:
+                raise PartError(f"unknown rotary pairing {pairing!r} (known: {', '.join(PAIRING)})")
+            if pairing == "adjacent":
+                self.rot_order = list(range(0, self.rot_dims, 2)) + list(range(1, self.rot_dims, 2)) \
+                    + list(range(self.rot_dims, self.rot))
         self.kv_size = 0 if self.shares_latent else self.R + self.rot
         self.g_size = self.nh if self.output_gate else 0
         # one product for everything that reads the mixer's input: [dq (or the queries themselves) | dkv | g]
@@ -122,7 +133,21 @@ class LatentAttention(Mixer):
             w["g"] = WeightSpec((self.nh, self.hidden))
         return w
 
+    def _reordered(self, w: torch.Tensor, groups: int) -> torch.Tensor:
+        """``w`` with the last ``rot_dim`` rows of each of its ``groups`` equal runs of rows in the kernels' order."""
+        if self.rot_order is None:
+            return w
+        w3 = w.view(groups, -1, w.shape[1])
+        head = w3.shape[1] - self.rot
+        order = torch.tensor(list(range(head)) + [head + i for i in self.rot_order], device=w.device)
+        return w3.index_select(1, order).reshape(w.shape)
+
     def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
+        tensors = dict(tensors)
+        queries = "uq" if self.Q > 0 else "q"
+        tensors[queries] = self._reordered(tensors[queries], self.nh)
+        if not self.shares_latent:
+            tensors["dkv"] = self._reordered(tensors["dkv"], 1)
         stacked = [tensors["dq" if self.Q > 0 else "q"]] + ([] if self.shares_latent else [tensors["dkv"]]) \
             + ([tensors["g"]] if self.output_gate else [])
         self.down.load(torch.cat(stacked, dim=0))

@@ -319,6 +319,74 @@ class HyperConnectionsBlock(Block):
         return delta
 
 
+@register("block", "sandwich_norm")
+class SandwichNormBlock(Block):
+    """A layer with a norm before AND after every sublayer:
+
+    ``x <- x + norm1b(mixer(norm1(x)))``, then ``x <- x + norm2b(feed_forward(norm2(x)))``.
+
+    It is a layer on ONE residual stream ``x [T, 1, hidden]`` (the model's ``streams`` is 1): a sublayer hands back sums
+    whose norm, weight and addition are left to the kernel that norms the stream for whoever reads it next, in this
+    layer or the one after, so a sublayer's two neighbouring norms are one pass over the row.
+
+    Parameters: ``hidden_size``, ``mixer``, ``feed_forward`` (None: the mixer alone), ``mixer_norm``,
+    ``feed_forward_norm`` (norms that offer ``forward_streams``), ``mixer_output_norm``, ``feed_forward_output_norm``
+    (RMS norms), and the weight-name prefixes of :class:`PreNormBlock` plus ``mixer_output_norm_prefix``,
+    ``feed_forward_output_norm_prefix``."""
+
+    def __init__(self, params, env: BuildEnv):
+        super().__init__(params, env)
+        self.require("hidden_size", "mixer", "mixer_norm", "mixer_output_norm")
+        self.hidden = int(params["hidden_size"])
+        self.feed_forward = self.feed_forward_norm = self.feed_forward_output_norm = None
+        self._prefixes = {}
+        self._one = None                                 # the stream's weight in what is read, mixed and written
+        self._weights = {}                               # output norms' weights as the kernel takes them
+
+        def part(kind, name):
+            made = build(kind, params[name], env)
+            self._prefixes[params.get(name + "_prefix", name + ".")] = made
+            return made
+        self.mixer = part("mixer", "mixer")
+        self.mixer_norm = part("norm", "mixer_norm")
+        self.mixer_output_norm = part("norm", "mixer_output_norm")
+        if params.get("feed_forward") is not None:
+            self.require("feed_forward_norm", "feed_forward_output_norm")
+            self.feed_forward = part("feed_forward", "feed_forward")
+            self.feed_forward_norm = part("norm", "feed_forward_norm")
+            self.feed_forward_output_norm = part("norm", "feed_forward_output_norm")
+        for norm in (self.mixer_output_norm, self.feed_forward_output_norm):
+            if norm is not None and type(norm) is not RMSNorm:
+                raise PartError("a norm on a sublayer's output must be an RMS norm here")
+
+    def sub_parts(self) -> Dict[str, Part]:
+        return dict(self._prefixes)
+
+    def finalize(self) -> None:
+        self._one = torch.ones(1, dtype=torch.float32, device=self.env.device)
+        self._weights = {id(n): n.weight.float().view(1, -1).contiguous()
+                         for n in (self.mixer_output_norm, self.feed_forward_output_norm) if n is not None}
+
+    def _sublayer(self, x, pending, norm, output_norm, run) -> StreamUpdate:
+        h = self.env.workspace.get("block.normed", (x.shape[0], self.hidden), self.env.dtype)
+        norm.forward_streams(x, self._one, h, pending=pending)
+        y = run(h)
+        if y.shape[0] != 1:
+            raise PartError("a sublayer of this block must hand back finished sums")
+        return StreamUpdate(Slices(y, weight=self._weights[id(output_norm)], eps=output_norm.eps), self._one,
+                            self._one.view(1, 1))
+
+    def forward(self, x: torch.Tensor, delta, step, cache: LayerCache):
+        if x.dim() != 3 or x.shape[1] != 1 or not (delta is None or isinstance(delta, StreamUpdate)):
+            raise PartError(f"this block keeps one residual stream [T, 1, hidden]; the model's residual is {tuple(x.shape)}")
+        delta = self._sublayer(x, delta, self.mixer_norm, self.mixer_output_norm,
+                               lambda h: self.mixer.forward(h, step, cache))
+        if self.feed_forward is not None:
+            delta = self._sublayer(x, delta, self.feed_forward_norm, self.feed_forward_output_norm,
+                                   lambda h: self.feed_forward.forward(h, step))
+        return delta
+
+
 class _Several(Part):
     """Parts of a block that share one weight-name prefix."""
 

@@ -12,6 +12,12 @@ with what differs between its kinds as parameters:
   ``a2.b``; ``tau``; the pair's inner width is ``rank``); ``"channel_token"``: the same pair, but
   ``exp(-exp(A_log[h]) * softplus(W_a2 (W_a1 h) + dt_bias))`` with a number ``A_log`` per head and ``dt_bias`` per
   head and channel;
+* decay ``{"kind": "exp_gates", "cap", "read_eps"}``: a matrix memory with exponential gates.  Per head and token a log
+  input gate ``i = cap tanh((W_i h + b_i) / cap)`` and a log forget gate ``f = logsigmoid(cap tanh((W_f h + b_f) / cap))``
+  (tensors ``i``, ``i.b``, ``f``, ``f.b``); with a running maximum ``m_t = max(f + m_{t-1}, i)`` from ``m = 0``,
+  ``a_t = exp(f + m_{t-1} - m_t)`` and ``u_t = exp(i - m_t) v_t``.  A vector ``n`` per head sums the keys as the state
+  sums ``k v^T``, and the read-out is divided by ``max(|n . q|, exp(-m_t)) + read_eps``.  ``n`` is the state's last column:
+  the values have one more column that is always 1.  ``m`` is state too;
 * ``delta_rule``: the state is corrected towards the value along the key, ``u_t = beta_t (v_t - S^T k_t)`` on
   the state already decayed, ``beta = sigmoid(W_b h)`` (tensor ``b``), and the read-out sees the correction;
   else ``u_t = v_t``;
@@ -25,8 +31,9 @@ with what differs between its kinds as parameters:
 * ``query_scale`` and ``key_scale`` multiply queries and keys (after rotation or unit norm);
 * ``qk_heads``: value head ``h`` reads query/key head ``h // (heads / qk_heads)``;
 * every head's read-out is divided by its root mean square (``norm_eps``), multiplied by a weight per coordinate
-  that the heads share (``norm_weight``: tensor ``norm``) or by nothing; with ``norm_over = "row"`` the heads are
-  normed together, over the whole row, with a weight per coordinate of the row;
+  that the heads share (``norm_weight``: tensor ``norm``) or by nothing; with ``norm_weight = "row"`` every head has
+  weights of its own (``norm [heads * value_dim]``); with ``norm_over = "row"`` the heads are normed together, over the
+  whole row, with a weight per coordinate of the row;
 * then it is multiplied by ``act(gate)`` (``gate = {"activation", "rank"}``: ``"silu"`` or ``"sigmoid"``; the gate is
   ``W_g h`` (tensor ``g``) or, with a ``rank``, ``W_g2 (W_g1 h)`` (tensors ``g1``, ``g2``)) and by ``output_scale``, and
   projected out (tensor ``o``).
@@ -50,6 +57,9 @@ from .base import BuildEnv, LayerCache, Mixer, PartError, Slices, WeightSpec, bu
 from .linear import Linear
 
 
+DECAY_KINDS = ("head", "head_token", "channel", "channel_token", "exp_gates")
+
+
 @register("mixer", "linear_recurrence")
 class LinearRecurrence(Mixer):
     """Parameters: ``hidden_size``, ``heads``, ``qk_heads`` (``heads``), ``key_dim``, ``value_dim``, ``decay``,
@@ -71,8 +81,9 @@ class LinearRecurrence(Mixer):
             raise PartError(f"head sizes {self.D}/{self.V} are not ones the kernel takes (keys up to 512)")
         decay = dict(p["decay"])
         self.decay_kind = decay.get("kind")
-        if self.decay_kind not in ops.recurrent.DECAY_MODES:
-            raise PartError(f"decay kind {self.decay_kind!r} is not known ({', '.join(ops.recurrent.DECAY_MODES)})")
+        if self.decay_kind not in DECAY_KINDS:
+            raise PartError(f"decay kind {self.decay_kind!r} is not known ({', '.join(DECAY_KINDS)})")
+        self.exp_gates = self.decay_kind == "exp_gates"
         self.decay_values = None
         self.tau, self.rank = 1.0, 0
         if self.decay_kind == "head":
@@ -83,6 +94,10 @@ class LinearRecurrence(Mixer):
             self.tau, self.rank = float(decay.get("tau", 1.0)), int(decay.get("rank") or 0)
             if not self.tau > 0 or self.rank <= 0:
                 raise PartError("a decay per channel needs a positive tau and the rank of its pair of products")
+        elif self.exp_gates:
+            self.cap, self.read_eps = float(decay.get("cap") or 0.0), float(decay.get("read_eps", 0.0))
+            if not self.cap > 0:
+                raise PartError("exponential gates need a positive cap")
         gate = dict(p.get("gate") or {})
         self.gate_act, self.gate_rank = gate.get("activation", "silu"), int(gate.get("rank") or 0)
         if self.gate_act not in ops.recurrent.GATE_ACTIVATIONS:
@@ -96,6 +111,8 @@ class LinearRecurrence(Mixer):
         self.qk = p.get("qk")
         if self.qk not in ops.recurrent.QK_MODES:
             raise PartError(f"qk {self.qk!r} is not known (rotate, unit, silu, None)")
+        if self.exp_gates and (self.delta_rule or self.qk == "silu" or p.get("norm_over", "head") != "head"):
+            raise PartError("exponential gates go with plain values, no delta rule and a norm per head")
         if self.qk == "silu" and self.taps > 0:
             raise PartError("a convolution activates queries, keys and values itself: qk \"silu\" is for none")
         self.position = None
@@ -112,9 +129,11 @@ class LinearRecurrence(Mixer):
             raise PartError("the delta rule is not linear in the key: key_scale must be 1")
         self.norm_eps = float(p["norm_eps"])
         self.norm_weight = bool(p.get("norm_weight", True))
+        self.norm_size = self.heads * self.V if "row" in (self.norm_over, p.get("norm_weight")) else self.V
         self.output_scale = float(p.get("output_scale", 1.0))
         self.qk_size, self.v_size = self.qk_heads * self.D, self.heads * self.V
-        # columns of the stacked projection: q | k | v | g (unless a narrow pair forms it) | beta | decay per head
+        # columns of the stacked projection: q | k | v | g (unless a narrow pair forms it) | beta | decay per head, or
+        # the two exponential gates
         self.cols = {"q": 0, "k": self.qk_size, "v": 2 * self.qk_size}
         total = 2 * self.qk_size + self.v_size
         if not self.gate_rank:
@@ -126,6 +145,9 @@ class LinearRecurrence(Mixer):
         if self.decay_kind == "head_token":
             self.cols["a"] = total
             total += self.heads
+        if self.exp_gates:
+            self.cols["i"], self.cols["f"] = total, total + self.heads
+            total += 2 * self.heads
         self.in_proj = Linear(env, total, self.hidden)
         self.out_proj = Linear(env, self.hidden, self.v_size)
         # narrow pairs: (first matrix, second matrix, inner width, outputs)
@@ -141,10 +163,12 @@ class LinearRecurrence(Mixer):
                 inner = -(-inner // 8) * 8           # rows of whole 16-byte runs, as the tensor-core products take them
             self.narrow = Linear(env, inner, self.hidden)
             self.wide = Linear(env, sum(n for _, _, _, n in self.pairs), inner)
-        self.state_floats = self.heads * self.D * self.V
+        self.VS = self.V + (1 if self.exp_gates else 0)          # columns of a head's state
+        self.matrix_floats = self.heads * self.D * self.VS
+        self.state_floats = self.matrix_floats + (self.heads if self.exp_gates else 0)
         self.conv_channels = 2 * self.qk_size + self.v_size
         self.conv_floats = max(self.taps - 1, 0) * self.conv_channels
-        self.norm_w = self.decay_const = self.dt_bias = self.conv_w = None
+        self.norm_w = self.decay_const = self.dt_bias = self.conv_w = self.i_bias = self.f_bias = None
 
     def parts(self):
         yield self
@@ -160,12 +184,15 @@ class LinearRecurrence(Mixer):
         for first, second, r, n in self.pairs:
             w.update({first: WeightSpec((r, H)), second: WeightSpec((n, r))})
         if self.norm_weight:
-            w["norm"] = WeightSpec((self.v_size if self.norm_over == "row" else self.V,), "norm")
+            w["norm"] = WeightSpec((self.norm_size,), "norm")
         if self.delta_rule:
             w["b"] = WeightSpec((self.heads, H))
         if self.decay_kind == "head_token":
             w.update({"a": WeightSpec((self.heads, H)), "A_log": WeightSpec((self.heads,), "bias"),
                       "dt_bias": WeightSpec((self.heads,), "bias")})
+        if self.exp_gates:
+            for n in ("i", "f"):
+                w.update({n: WeightSpec((self.heads, H)), n + ".b": WeightSpec((self.heads,), "bias")})
         if self.decay_kind == "channel":
             w["a2.b"] = WeightSpec((self.heads * self.D,), "bias")
         if self.decay_kind == "channel_token":
@@ -184,6 +211,9 @@ class LinearRecurrence(Mixer):
             stacked.append(tensors["b"])
         if self.decay_kind == "head_token":
             stacked.append(tensors["a"])
+        if self.exp_gates:
+            stacked += [tensors["i"], tensors["f"]]
+            self.i_bias, self.f_bias = (tensors[n].float().contiguous() for n in ("i.b", "f.b"))
         if self.decay_kind in ("head_token", "channel_token"):
             self.decay_const = tensors["A_log"].float().contiguous()
             self.dt_bias = tensors["dt_bias"].float().contiguous()
@@ -225,7 +255,7 @@ class LinearRecurrence(Mixer):
             raise PartError("a recurrent mixer needs a state slot per request")
         proj = self.in_proj.forward(h, "linrec.proj", "float32")
         rows = cache.state.view(torch.float32)
-        state = rows[:, :self.state_floats].unflatten(1, (self.heads, self.D, self.V))
+        state = rows[:, :self.matrix_floats].unflatten(1, (self.heads, self.D, self.VS))
         c = self.cols
         if self.taps > 0:
             conv_state = rows[:, self.state_floats:self.state_floats + self.conv_floats] \
@@ -246,10 +276,20 @@ class LinearRecurrence(Mixer):
                 decay_channel = wide[:, :at]
             if self.gate_rank:
                 gate = wide[:, at:]
-        y = ws.get("linrec.y", (T, self.v_size), torch.float32)
+        decay, decay_head, write_gate, floor = self.decay_kind, None, None, None
+        if "a" in c:
+            decay_head = proj[:, c["a"]:c["a"] + self.heads]
+        if self.exp_gates:
+            decay, decay_head = "head_ready", proj[:, c["f"]:c["f"] + self.heads]
+            write_gate = proj[:, c["i"]:c["i"] + self.heads]
+            floor = ws.get("linrec.floor", (T, self.heads), torch.float32)
+            ops.exp_gates(write_gate, decay_head, self.i_bias, self.f_bias, self.cap,
+                          rows[:, self.matrix_floats:self.state_floats], step.seq_start, step.positions,
+                          step.state_slots, floor, S)
+        y = ws.get("linrec.y", (T, self.heads * self.VS), torch.float32)
         ops.linear_scan(q, k, v, y, state, step.seq_start, step.positions, step.state_slots, S, self.heads,
-                        self.qk_heads, self.D, self.V, self.decay_kind, decay_channel=decay_channel, tau=self.tau,
-                        decay_head=proj[:, c["a"]:c["a"] + self.heads] if "a" in c else None,
+                        self.qk_heads, self.D, self.V, decay, decay_channel=decay_channel, tau=self.tau,
+                        decay_head=decay_head, write_gate=write_gate, unit_column=self.exp_gates,
                         decay_const=self.decay_const, dt_bias=self.dt_bias,
                         beta=proj[:, c["b"]:c["b"] + self.heads] if self.delta_rule else None, qk=self.qk,
                         cos_sin=self.position.rotation_for(step)[0] if self.position is not None else None,
@@ -257,7 +297,7 @@ class LinearRecurrence(Mixer):
         gated = ws.get("linrec.gated", (T, self.v_size), self.env.dtype)
         heads, V = (1, self.v_size) if self.norm_over == "row" else (self.heads, self.V)
         ops.head_norm_gate(y, gate, self.norm_w, self.norm_eps, gated, heads, V, out_scale=self.output_scale,
-                           activation=self.gate_act)
+                           activation=self.gate_act, floor=floor, floor_eps=self.read_eps if self.exp_gates else 0.0)
         return self.out_proj.forward(gated, "linrec.o", "delta", into=into)
 
 

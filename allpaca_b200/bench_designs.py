@@ -1,9 +1,11 @@
 """Prefill and decode throughput of one design beside the dense Llama decoder of equal size,
 with the time of every kind of kernel in a step:
 
-    python bench.py --design viresun|bivatar|lazolix|gezozen|boketar [--design-size small|base|wide]
+    python bench.py --design viresun|bivatar|lazolix|gezozen|boketar|merusun [--design-size small|base|wide]
 
-Boketar runs beside the Gezozen decoder (the closest existing model: softmax attention beside a linear attention, a
+Merusun runs beside the Gezozen decoder (the closest existing model: a recurrent mixer with fixed-size state, windowed
+softmax attention, routed experts with a shared expert in every layer) and the Llama decoder.  Boketar runs beside the
+Gezozen decoder (the closest existing model: softmax attention beside a linear attention, a
 delta rule with short convolutions) and the Llama decoder.  Gezozen runs beside the Viresun decoder (the closest existing model: windowed attention, a recurrent mixer
 with fixed-size state, routed experts) and the Llama decoder.  Lazolix runs beside two models: the Bivatar decoder reduced to its latent layers (the closest existing
 mixer) and the Llama decoder.  All models have random bfloat16 weights drawn on the device, the same width, heads, head size,
@@ -130,6 +132,25 @@ def boketar_config(size: str) -> dict:
                        {"type": "channel_delta", "mixer": delta, "mlp": dense}, {"type": "parallel", "mixer": pair, "mlp": dense}]}
 
 
+def merusun_config(size: str) -> dict:
+    """Four layers, all with squared-ReLU experts routed among the best half of four groups and a shared expert: a matrix
+    memory; windowed latent attention with a rotated key part; windowed attention; windowed attention on the third
+    layer's keys and values."""
+    W, H, G, D, ff, E, top, eff, window = SIZES[size][:9]
+    R, _, nope, rot, vd, _ = LATENT_SIZES[size]
+    memory = {"heads": H, "dim": D, "vdim": D, "gate_cap": 15.0}
+    latent = {"heads": H, "dim": nope, "rot_dim": rot, "vdim": vd, "kv_rank": R, "scale": (nope + rot) ** -0.5,
+              "mask": {"size": window}, "rot": {"base": 10000.0, "dims": rot}}
+    attn = {"heads": H, "kv_heads": G, "dim": D, "vdim": D, "scale": D ** -0.5, "mask": {"size": window}}
+    moe = {"kind": "moe", "expert": {"ff": eff}, "shared": {"ff": eff},
+           "router": {"experts": E, "top": top, "scale": 2.5, "groups": {"count": 4, "keep": 2}}}
+    return {"architecture": "Merusun", "vocab": VOCAB, "width": W, "norm": {"eps": 1e-6}, "embedding": {"scale": 8.0},
+            "layers": [{"type": "mlstm", "mixer": memory, "mlp": moe},
+                       {"type": "latent_attention", "mixer": latent, "mlp": moe},
+                       {"type": "attention", "mixer": attn, "mlp": moe},
+                       {"type": "attention", "mixer": dict(attn, kv_from=2), "mlp": moe}]}
+
+
 def bivatar_latent_config(size: str) -> dict:
     """The Bivatar decoder with latent layers only (the windowed layer left out): what Lazolix runs beside."""
     raw = bivatar_config(size)
@@ -141,6 +162,9 @@ def bivatar_latent_config(size: str) -> dict:
 
 
 DESIGNS = {
+    "merusun": (merusun_config, "norms before and after every sublayer; matrix memory, windowed latent attention, windowed "
+                                "attention, windowed attention on the third layer's keys and values; squared-ReLU experts "
+                                "routed among groups with a shared expert in every layer"),
     "boketar": (boketar_config, "hyper-connections over 4 residual streams; delta rule with a decay per key channel, "
                                 "windowed attention with short convolutions and a sink beside lightning attention, "
                                 "the same two again; dense feed-forwards"),
@@ -297,6 +321,13 @@ def run(design: str, size: str, steps: int, warmup: int, batch: int, context: in
     if design == "boketar":
         sizes = {k: v for k, v in sizes.items() if k in ("width", "heads", "kv_heads", "head_dim", "ff", "window")}
         sizes.update({"lightning_heads": max(sizes["heads"] // 2, 1), "streams": STREAMS, "narrow": NARROW})
+        others.insert(0, ("gezozen", gezozen_config(size)))
+    if design == "merusun":
+        sizes = {k: v for k, v in sizes.items() if k in ("width", "heads", "kv_heads", "head_dim", "experts", "top",
+                                                         "expert_ff", "window")}
+        R, _, nope, rot, vd, _ = LATENT_SIZES[size]
+        sizes.update({"kv_rank": R, "dim": nope, "rot_dim": rot, "vdim": vd, "shared_ff": sizes["expert_ff"], "groups": 4,
+                      "keep": 2})
         others.insert(0, ("gezozen", gezozen_config(size)))
     if design == "gezozen":
         sizes = {k: v for k, v in sizes.items() if k in ("width", "heads", "kv_heads", "head_dim", "experts", "top",

@@ -427,6 +427,10 @@ def bench_stream(args) -> dict:
     chosen, share = torch.empty(T, top, dtype=torch.int32, device=dev), torch.empty(T, top, device=dev)
     cases["moe_route_rows"] = (lambda i: ops.moe_route_rows(hb[i % len(hb)], router, correction, chosen, share,
                                                             "softmax_all"), T * H * 2 + E * H * 2)
+    if E % 4 == 0 and top <= E // 2:
+        cases["moe_route_rows, two groups of four"] = (
+            lambda i: ops.moe_route_rows(hb[i % len(hb)], router, None, chosen, share, "softmax_scores", groups=4, keep=2),
+            T * H * 2 + E * H * 2)
     res = {"rows": T, "width": H, "streams": K + 1, "ff": F, "seqs": nseq, "experts": E, "top": top}
     for name, (fn, nbytes) in cases.items():
         us = _time(fn, args.iters, args.warmup, not args.no_graph)
@@ -440,8 +444,9 @@ def bench_recurrent(args) -> dict:
     per head and with one per channel) on ``--seqs`` sequences of ``--rows`` rows each, beside
     the state-space recurrence of the same state size (``ssm_scan``); and the norm after a gated sum beside
     ``add_rmsnorm`` and ``norm_residual`` on the same rows, the norm behind hyper-connections of ``--streams`` residual
-    streams (with one pending slice, and with two that are normed on their own), and the causal convolution, each
-    beside the bytes it must move."""
+    streams (with one pending slice, and with two that are normed on their own), the same kernel between two sublayers of
+    a layer with norms before and after each, the causal convolution, and a matrix memory's exponential gates, recurrence
+    and read-out, each beside the bytes it must move."""
     from allpaca_b200 import ops
     n, S, H, D, V, W = args.rows, max(1, args.seqs), args.heads, args.dim, args.vdim, args.width
     T = n * S
@@ -515,6 +520,25 @@ def bench_recurrent(args) -> dict:
     cases[f"stream_norm, {N} streams, two normed slices"] = (
         lambda i: ops.stream_norm(streams[i % sc], win, w32, 1e-6, copy, delta=pend2[i % sc], out_w=wout, mix=wmix,
                                   slice_bias=sb, slice_weight=sw, slice_eps=1e-6), T * W * (8 * N + 10))
+    one, one1 = torch.ones(1, device=dev), torch.ones(1, 1, device=dev)
+    single = [x.view(T, 1, W) for x in xs]
+    cases["stream_norm, 1 stream, a normed slice"] = (
+        lambda i: ops.stream_norm(single[i % wc], one, w32, 1e-6, copy, delta=ds[i % wc], out_w=one, mix=one1,
+                                  slice_weight=sw[:1], slice_eps=1e-6), T * W * 14)
+    gi = [rnd(T, 2 * H) for _ in range(copies)]
+    top, floor = torch.zeros(S, H, device=dev), torch.empty(T, H, device=dev)
+    cases["exp_gates"] = (lambda i: ops.exp_gates(gi[i % copies][:, :H], gi[i % copies][:, H:], dt_bias, dt_bias, 15.0, top,
+                                                  seq_start, positions, slots, floor, S), T * H * 20)
+    ym, sm = torch.empty(T, H * (V + 1), device=dev), torch.zeros(S, H, D, V + 1, device=dev)
+    keep, write = torch.sigmoid(3.0 + rnd(T, H)), torch.rand(T, H, device=dev)
+    cases["la_scan matrix memory"] = (
+        lambda i: ops.linear_scan(q[i % copies], k[i % copies], v[i % copies], ym, sm, seq_start, positions, slots, S, H, H, D, V,
+                                  "head_ready", workspace=ws, decay_head=keep, write_gate=write, unit_column=True), io)
+    yms = [rnd(T, H * (V + 1)) for _ in range(copies)]
+    nwh, ones = torch.ones(H * V, device=dev), torch.ones(T, H, device=dev)
+    cases["head_norm_gate, over a denominator"] = (
+        lambda i: ops.head_norm_gate(yms[i % copies], gate[i % copies], nwh, 1e-6, out, H, V, activation="sigmoid", floor=ones,
+                                     floor_eps=1e-6), T * H * V * 10)
     C = 2 * H * D + H * V
     cc = max(2, int(math.ceil(300e6 / (T * C * 4))))
     cin = [rnd(T, C) for _ in range(cc)]

@@ -422,7 +422,12 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
                 } else if (n < N) {
 #pragma unroll
                     for (int jj = 0; jj < 32; ++jj) {
-                        if (c + jj < cols) out[(size_t)(m0 + c + jj) * ldc + n] = ap_from_float<TO>(__uint_as_float(v[jj]));
+                        float x = __uint_as_float(v[jj]);
+                        if (act == 2) {                       // no gate, the square of relu
+                            x = fmaxf(x, 0.f);
+                            x *= x;
+                        }
+                        if (c + jj < cols) out[(size_t)(m0 + c + jj) * ldc + n] = ap_from_float<TO>(x);
                     }
                 }
             }
@@ -553,7 +558,8 @@ static int launch_pair(const CUtensorMap& mw, const CUtensorMap& ma, void* out, 
 
 // The product on pairs of SMs (see gemm_tc_pair_kernel), for products with many rows.
 //   pairs == 0: out[M, N] = a * w^T for w [N, K].
-//   pairs != 0: w [N, K] has gate and up rows alternating; out[M, N/2] = silu(gate) * up.
+//   pairs 1, 2: w [N, K] has gate and up rows alternating; out[M, N/2] = silu(gate) * up (1) or gelu_tanh(gate) * up (2).
+//   pairs == 3: as 0, with the square of relu on the sums.
 //   scratch: null, or a zeroed buffer of ap_gemm_tc_pair_scratch_bytes() bytes that belongs to one
 //   stream (few tiles of a long K are then shared among several pairs; the kernel leaves the flags
 //   at its head zero again).  The persistent kernel's scratch buffer serves both.
@@ -568,9 +574,10 @@ AP_EXPORT int ap_gemm_tc_pair(const void* a, const void* w, void* out, int out_d
     AP_REQUIRE(K % 8 == 0 && lda % 8 == 0 && ldw % 8 == 0,
                "gemm_tc_pair: K=%d and the leading dimensions must be multiples of 8 (16-byte rows for TMA)", K);
     AP_REQUIRE(((uintptr_t)a & 15) == 0 && ((uintptr_t)w & 15) == 0, "gemm_tc_pair: operands must be 16-byte aligned");
+    AP_REQUIRE(pairs >= 0 && pairs <= 3, "gemm_tc_pair: pairs is 0, 1 (silu), 2 (gelu_tanh) or 3 (no gate, relu2)");
+    const int act = pairs == 3 ? 2 : (pairs == 2 ? 1 : 0);
+    if (pairs == 3) pairs = 0;
     AP_REQUIRE(!pairs || N % 2 == 0, "gemm_tc_pair: gate and up rows alternate, so the weight has an even number of rows");
-    AP_REQUIRE(pairs >= 0 && pairs <= 2, "gemm_tc_pair: pairs is 0, 1 (silu) or 2 (gelu_tanh)");
-    const int act = pairs == 2 ? 1 : 0;
     AP_REQUIRE(lda >= K && ldw >= K && ldc >= (pairs ? N / 2 : N), "gemm_tc_pair: a leading dimension is below its row length");
     AP_REQUIRE(out_dtype == AP_F32 || out_dtype == AP_BF16, "gemm_tc_pair: unknown output dtype %d", out_dtype);
     // token tiles of at most 256 rows, evenly filled; a tile's width is a multiple of 32 (each CTA
@@ -586,8 +593,8 @@ AP_EXPORT int ap_gemm_tc_pair(const void* a, const void* w, void* out, int out_d
                    : launch_pair<bf16, true>(mw, ma, out, M, N, K, ldc, bn, tiles_m, scratch, scratch_bytes, act, stream);
     }
     return out_dtype == AP_F32
-               ? launch_pair<float, false>(mw, ma, out, M, N, K, ldc, bn, tiles_m, scratch, scratch_bytes, 0, stream)
-               : launch_pair<bf16, false>(mw, ma, out, M, N, K, ldc, bn, tiles_m, scratch, scratch_bytes, 0, stream);
+               ? launch_pair<float, false>(mw, ma, out, M, N, K, ldc, bn, tiles_m, scratch, scratch_bytes, act, stream)
+               : launch_pair<bf16, false>(mw, ma, out, M, N, K, ldc, bn, tiles_m, scratch, scratch_bytes, act, stream);
 }
 
 // Whether this kernel is the one to use for a product of many rows.  Measured against the

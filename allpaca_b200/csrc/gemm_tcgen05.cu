@@ -52,7 +52,7 @@ template <int BN, bool CLUSTER = false> struct TileCfg {
 };
 
 // What the epilogue does with the finished sums.
-//   EPI_PLAIN     out[m, n] = sum                                  (32-bit or bfloat16 out)
+//   EPI_PLAIN     out[m, n] = sum, or an activation of it          (32-bit or bfloat16 out)
 //   EPI_PAIRS     the weight's rows alternate gate, up, gate, up ...; the sums of row 2i and 2i+1
 //                 become out[m, i] = silu(gate) * up (out is [M, N/2]), so that the gated
 //                 activation of a decode step needs no kernel of its own
@@ -82,7 +82,7 @@ struct EpiArgs {
     long long ldxb;
     float* ss_out;           // EPI_RESIDUAL: [M][ss_out_parts]
     int ss_out_parts;
-    int act;                 // EPI_PAIRS: the gate's activation (see gated())
+    int act;                 // EPI_PAIRS: the gate's activation (see gated()); EPI_PLAIN: the sums' (see activated())
     // EPI_ROPE
     bf16* q_out;             // [M][nh * hd]
     bf16* cache;             // one layer's pages [page][2][nkv][P][hd], or nullptr: store no K, V
@@ -133,6 +133,14 @@ __device__ __forceinline__ float gated(float gate, float up, int act) {
         return 0.5f * gate * (1.0f + th) * up;
     }
     return __fdividef(gate, 1.0f + __expf(-gate)) * up;
+}
+// A finished sum on its way out of a product without gates: act 2: the square of relu; else as it is.
+__device__ __forceinline__ float activated(float v, int act) {
+    if (act == 2) {
+        v = fmaxf(v, 0.f);
+        v *= v;
+    }
+    return v;
 }
 // the four epilogue warps among themselves (barrier 1; barrier 0 is __syncthreads)
 __device__ __forceinline__ void epilogue_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
@@ -395,7 +403,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constant
 #pragma unroll
                     for (int j = 0; j < 16; ++j) {
                         const int m = m0 + c + j;
-                        if (m < M) out[(size_t)m * ldc + n] = ap_from_float<TO>(__uint_as_float(v[j]) * inv_s[c + j]);
+                        if (m < M) out[(size_t)m * ldc + n] = ap_from_float<TO>(activated(__uint_as_float(v[j]) * inv_s[c + j], ea.act));
                     }
                 }
             }
@@ -524,7 +532,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constant
                     float sum = 0.f;
                     for (int s = 0; s < S; ++s) sum += reduce[(s * BN + c) * band + i];   // slices in order
                     const int n = n0 + first + i;
-                    if (n < N) out[(size_t)(m0 + c) * ldc + n] = ap_from_float<TO>(sum * inv_s[c]);
+                    if (n < N) out[(size_t)(m0 + c) * ldc + n] = ap_from_float<TO>(activated(sum * inv_s[c], ea.act));
                 }
             }
         }
@@ -809,7 +817,7 @@ static int gemm_tc_run(const void* a, const void* w, void* out, int out_dtype, i
 // reduce != 0: the K slices add up inside a thread-block cluster and `out` is the finished
 // matrix (nsplit <= 8, M <= 256); else slice z writes 32-bit partial sums at out + z * split_stride.
 // epi: what becomes of the finished sums (nsplit == 1, or reduce):
-//   0  out[M, N] = sums, 32-bit or bfloat16;
+//   0  out[M, N] = sums, 32-bit or bfloat16 (512: the square of their relu; finished sums only);
 //   1  w's rows alternate gate and up, out[M, N/2] = silu(gate) * up (bfloat16, M <= 256);
 //   2  out is the 32-bit residual [M, N] and is added to; xb [M, ldxb] receives its bfloat16
 //      copy and ss_out [M, ap_gemm_tc_residual_parts(N, nsplit)] partial sums of squares of the
@@ -826,10 +834,12 @@ AP_EXPORT int ap_gemm_tc(const void* a, const void* w, void* out, int out_dtype,
     AP_REQUIRE(K % 8 == 0 && lda % 8 == 0 && ldw % 8 == 0,
                "gemm_tc: K=%d and the leading dimensions must be multiples of 8 (16-byte rows for TMA)", K);
     AP_REQUIRE(((uintptr_t)a & 15) == 0 && ((uintptr_t)w & 15) == 0, "gemm_tc: operands must be 16-byte aligned");
-    // EPI_PAIRS: the gate's activation rides above the code (gemm_tc_run takes the two apart)
+    // EPI_PAIRS, EPI_PLAIN: the activation rides above the code (gemm_tc_run takes the two apart)
     AP_REQUIRE((epi & 0xff) == EPI_PLAIN || (epi & 0xff) == EPI_PAIRS || (epi & 0xff) == EPI_RESIDUAL,
                "gemm_tc: unknown epilogue %d", epi & 0xff);
-    AP_REQUIRE((epi >> 8) == 0 || ((epi >> 8) == 1 && (epi & 0xff) == EPI_PAIRS), "gemm_tc: unknown activation %d", epi >> 8);
+    AP_REQUIRE((epi >> 8) == 0 || ((epi >> 8) == 1 && (epi & 0xff) == EPI_PAIRS) || ((epi >> 8) == 2 && (epi & 0xff) == EPI_PLAIN),
+               "gemm_tc: unknown activation %d", epi >> 8);
+    AP_REQUIRE((epi >> 8) != 2 || nsplit == 1 || reduce, "gemm_tc: an activation takes finished sums");
     return gemm_tc_run(a, w, out, out_dtype, M, N, K, lda, ldw, ldc, nsplit, split_stride, reduce, epi, ss_in,
                        ss_in_parts, inv_width, eps, xb, ldxb, ss_out, ss_out_parts, nullptr, stream);
 }
@@ -839,7 +849,7 @@ static int gemm_tc_run(const void* a, const void* w, void* out, int out_dtype, i
                        int reduce, int epi, const float* ss_in, int ss_in_parts, float inv_width, float eps,
                        void* xb, long long ldxb, float* ss_out, int ss_out_parts, const EpiArgs* rope,
                        cudaStream_t stream) {
-    const int act = epi >> 8;                               // the gate's activation of EPI_PAIRS
+    const int act = epi >> 8;                               // the activation of EPI_PAIRS or EPI_PLAIN
     epi &= 0xff;
     const bool pairs = epi == EPI_PAIRS;
     AP_REQUIRE(lda >= K && ldw >= K && ldc >= (pairs ? N / 2 : N), "gemm_tc: a leading dimension is below its row length");
@@ -1288,7 +1298,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const __gr
                 } else if (n < N) {
 #pragma unroll
                     for (int jj = 0; jj < 32; ++jj) {
-                        if (c + jj < cols) out[(size_t)(m0 + c + jj) * ldc + n] = ap_from_float<TO>(__uint_as_float(v[jj]));
+                        if (c + jj < cols) out[(size_t)(m0 + c + jj) * ldc + n] = ap_from_float<TO>(activated(__uint_as_float(v[jj]), act));
                     }
                 }
             }
@@ -1365,7 +1375,7 @@ AP_EXPORT long long ap_gemm_tc_persistent_scratch_bytes(void) {
 // The persistent kernel (see gemm_tc_persistent_kernel), for products with more than 64 rows.
 //   pairs == 0: out[M, N] = a * w^T for w [N, K].
 //   pairs != 0: w [N, K] has gate and up rows alternating; out[M, N/2] = silu(gate) * up (pairs 1) or
-//               gelu_tanh(gate) * up (pairs 2).
+//               gelu_tanh(gate) * up (pairs 2).  pairs 3 is pairs 0 with the square of relu on the sums.
 //   scratch: null, or ap_gemm_tc_persistent_scratch_bytes() bytes (see there).
 AP_EXPORT int ap_gemm_tc_persistent(const void* a, const void* w, void* out, int out_dtype, int M, int N, int K,
                                     long long lda, long long ldw, long long ldc, int pairs, void* scratch,
@@ -1375,9 +1385,10 @@ AP_EXPORT int ap_gemm_tc_persistent(const void* a, const void* w, void* out, int
     AP_REQUIRE(K % 8 == 0 && lda % 8 == 0 && ldw % 8 == 0,
                "gemm_tc: K=%d and the leading dimensions must be multiples of 8 (16-byte rows for TMA)", K);
     AP_REQUIRE(((uintptr_t)a & 15) == 0 && ((uintptr_t)w & 15) == 0, "gemm_tc: operands must be 16-byte aligned");
+    AP_REQUIRE(pairs >= 0 && pairs <= 3, "gemm_tc: pairs is 0, 1 (silu), 2 (gelu_tanh) or 3 (no gate, relu2)");
+    const int act = pairs == 3 ? 2 : (pairs == 2 ? 1 : 0);
+    if (pairs == 3) pairs = 0;
     AP_REQUIRE(!pairs || N % 2 == 0, "gemm_tc: gate and up rows alternate, so the weight has an even number of rows");
-    AP_REQUIRE(pairs >= 0 && pairs <= 2, "gemm_tc: pairs is 0, 1 (silu) or 2 (gelu_tanh)");
-    const int act = pairs == 2 ? 1 : 0;
     AP_REQUIRE(lda >= K && ldw >= K && ldc >= (pairs ? N / 2 : N), "gemm_tc: a leading dimension is below its row length");
     AP_REQUIRE(out_dtype == AP_F32 || out_dtype == AP_BF16, "gemm_tc: unknown output dtype %d", out_dtype);
     // token tiles: as many as tiles of the full width (128 for up to 128 rows, else 256) would

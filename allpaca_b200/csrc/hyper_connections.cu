@@ -12,8 +12,11 @@
 // copies of the embedding row, which is then the pending result).  Without a pending result the streams stay as they
 // are.  With chosen rows only those are produced and the streams are left alone: the model's last norm.
 //
+// ONE stream with one normed slice is a layer with a norm before and after each sublayer, and has a kernel of its own.
+//
 // All 32-bit up to the store of `out`.  One CTA per row; sums over a row are formed in a fixed order that depends on
-// the width alone, so a row has the same bits in any batch.
+// the width alone (for the one stream also on whether the step has few rows or many), so a row has the same bits in any
+// such batch.
 #include "common.cuh"
 
 #define HC_MAX_STREAMS 32
@@ -254,6 +257,62 @@ __global__ void __launch_bounds__(ONE && NS <= 4 ? 1024 : 512) stream_norm_kerne
     }
 }
 
+// One stream, one pending slice over its own root mean square:
+//   x <- mix x + out_w (scale rmsnorm(delta) slice_w)        out = rmsnorm(in_w x) w
+// A thread holds PV runs of four columns of both rows in registers through the two sums over the row.
+template <int PV, typename TO>
+__global__ void __launch_bounds__(512) one_stream_norm_kernel(const StreamNormArgs A, TO* __restrict__ out) {
+    __shared__ float first_s[32], second_s[32];
+    ap_pdl_trigger();
+    const float mix = A.mix[0], out_w = A.out_w[0] * A.slice_scale, in_w = A.in_w[0];
+    ap_pdl_wait();
+    const int H = A.H;
+    const size_t t = A.rows ? (size_t)A.rows[blockIdx.x] : (size_t)blockIdx.x;
+    float* xr = A.x + t * H;
+    const float* dr = A.delta + t * H;
+    float4 d[PV], x[PV];
+#pragma unroll
+    for (int j = 0; j < PV; ++j) {
+        const int c = (j * (int)blockDim.x + (int)threadIdx.x) * 4;
+        d[j] = x[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (c < H) {
+            d[j] = *reinterpret_cast<const float4*>(dr + c);
+            x[j] = *reinterpret_cast<const float4*>(xr + c);
+        }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < PV; ++j) ss = fmaf(d[j].x, d[j].x, fmaf(d[j].y, d[j].y, fmaf(d[j].z, d[j].z, fmaf(d[j].w, d[j].w, ss))));
+    ss = ap_block_sum(ss, first_s);
+    const float f = out_w / sqrtf(ss / (float)H + A.slice_eps);
+    ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < PV; ++j) {
+        const int c = (j * (int)blockDim.x + (int)threadIdx.x) * 4;
+        if (c < H) {
+            const float4 w = *reinterpret_cast<const float4*>(A.slice_w + c);
+            x[j].x = fmaf(mix, x[j].x, f * d[j].x * w.x);
+            x[j].y = fmaf(mix, x[j].y, f * d[j].y * w.y);
+            x[j].z = fmaf(mix, x[j].z, f * d[j].z * w.z);
+            x[j].w = fmaf(mix, x[j].w, f * d[j].w * w.w);
+            if (A.update) *reinterpret_cast<float4*>(xr + c) = x[j];
+        }
+        x[j].x *= in_w; x[j].y *= in_w; x[j].z *= in_w; x[j].w *= in_w;
+        ss = fmaf(x[j].x, x[j].x, fmaf(x[j].y, x[j].y, fmaf(x[j].z, x[j].z, fmaf(x[j].w, x[j].w, ss))));
+    }
+    ss = ap_block_sum(ss, second_s);
+    const float inv = 1.0f / sqrtf(ss / (float)H + A.eps);
+#pragma unroll
+    for (int j = 0; j < PV; ++j) {
+        const int c = (j * (int)blockDim.x + (int)threadIdx.x) * 4;
+        if (c < H) {
+            const float4 w = *reinterpret_cast<const float4*>(A.w + c);
+            const float v[4] = {x[j].x * inv * w.x, x[j].y * inv * w.y, x[j].z * inv * w.z, x[j].w * inv * w.w};
+            hc_store<4>(out + (size_t)blockIdx.x * H + c, v);
+        }
+    }
+}
+
 AP_EXPORT int ap_stream_norm(float* x, const int* rows, int R, const float* delta, int S, long long slice_stride,
                              const float* slice_bias, const float* slice_w, float slice_eps, float slice_scale,
                              const float* out_w, const float* mix, const float* in_w, const float* w, float eps,
@@ -278,6 +337,27 @@ AP_EXPORT int ap_stream_norm(float* x, const int* rows, int R, const float* delt
     A.slice_bias = slice_bias; A.slice_w = slice_w; A.slice_eps = slice_eps; A.slice_scale = slice_scale;
     A.out_w = out_w; A.mix = mix; A.in_w = in_w; A.w = w; A.eps = eps; A.update = (update && delta) ? 1 : 0;
     A.streams = streams; A.H = H;
+    AP_REQUIRE(out_dtype == AP_F32 || out_dtype == AP_BF16, "stream_norm: unknown dtype %d", out_dtype);
+    if (streams == 1 && vec && delta && S == 1 && slice_w && !slice_bias && mix && H <= 16384) {
+        // runs of four columns to a thread: in a step of many rows more of them, so that an SM holds many rows at once
+        const int runs = H / 4, want = R >= 4 * 148 ? 128 : 512;
+        int pv = 1;
+        while (pv < 8 && (runs + pv - 1) / pv > want) pv *= 2;
+        const int nt = ((runs + pv - 1) / pv + 31) / 32 * 32;
+#define LAUNCH_ONE(PV)                                                                                              \
+        do {                                                                                                        \
+            if (out_dtype == AP_F32)                                                                                \
+                AP_CHECK_PDL_LAUNCH("stream_norm", ap_launch_pdl(one_stream_norm_kernel<PV, float>, dim3((unsigned)R), dim3(nt), 0, stream, A, (float*)out)); \
+            else                                                                                                    \
+                AP_CHECK_PDL_LAUNCH("stream_norm", ap_launch_pdl(one_stream_norm_kernel<PV, bf16>, dim3((unsigned)R), dim3(nt), 0, stream, A, (bf16*)out));   \
+        } while (0)
+        if (pv == 1) LAUNCH_ONE(1);
+        else if (pv == 2) LAUNCH_ONE(2);
+        else if (pv == 4) LAUNCH_ONE(4);
+        else LAUNCH_ONE(8);
+#undef LAUNCH_ONE
+        return AP_OK;
+    }
 #define LAUNCH(N, V, ONE, TO)                                                                                       \
     do {                                                                                                            \
         auto kern = stream_norm_kernel<N, V, ONE, TO>;                                                                  \
@@ -289,7 +369,6 @@ AP_EXPORT int ap_stream_norm(float* x, const int* rows, int R, const float* delt
     } while (0)
 #define LAUNCH_T(N, V, ONE) do { if (out_dtype == AP_F32) LAUNCH(N, V, ONE, float); else LAUNCH(N, V, ONE, bf16); } while (0)
 #define LAUNCH_V(N) do { if (one) LAUNCH_T(N, 4, true); else if (vec) LAUNCH_T(N, 4, false); else LAUNCH_T(N, 1, false); } while (0)
-    AP_REQUIRE(out_dtype == AP_F32 || out_dtype == AP_BF16, "stream_norm: unknown dtype %d", out_dtype);
     switch (streams) {
         case 1: LAUNCH_V(1); break;
         case 2: LAUNCH_V(2); break;

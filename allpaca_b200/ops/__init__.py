@@ -61,6 +61,18 @@ def _pairs_code(pairs) -> int:
     raise KernelError(f"the gated epilogue of a product knows silu and gelu_tanh, not {pairs!r}")
 
 
+EPILOGUE_ACTIVATIONS = {None: 0, "relu2": 2}       # of a product without gates, in its own epilogue
+
+
+def _epilogue_code(pairs, activation) -> int:
+    """``pairs`` (see :func:`_pairs_code`), or an ``activation`` of a product without gates."""
+    if activation is None:
+        return _pairs_code(pairs)
+    if pairs or activation not in EPILOGUE_ACTIVATIONS:
+        raise KernelError(f"the epilogue of a product without gates knows relu2, not {activation!r}")
+    return 3
+
+
 def embed_gather(tokens: torch.Tensor, table: torch.Tensor, x: torch.Tensor, scale: float = 1.0) -> None:
     """``x[t] = table[tokens[t]] * scale`` into the 32-bit residual stream ``x [T,H]``."""
     _check(tokens, "tokens", torch.int32, 1)
@@ -292,7 +304,8 @@ def _scale_args(scale: Optional[RowScale], M: int):
 
 
 def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, nsplit: int = 1,
-            reduce: bool = False, pairs: bool = False, scale: Optional[RowScale] = None) -> None:
+            reduce: bool = False, pairs: bool = False, scale: Optional[RowScale] = None,
+            activation: Optional[str] = None) -> None:
     """bfloat16 ``a[M,K] @ w[N,K]^T`` on the tcgen05 tensor cores.
 
     ``nsplit`` K slices run as separate CTAs.  With ``reduce`` they add up inside a
@@ -300,11 +313,13 @@ def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, nsplit: int = 1
     ``[M,N]`` in bfloat16 or float32; without it ``out`` is float32 ``[nsplit, M, N]`` partial
     sums (``[M,N]`` for ``nsplit == 1``).  ``pairs`` (at most 256 rows, finished sums, bfloat16
     out): the rows of ``w`` alternate gate and up, and ``out[M,N/2] = silu(gate) * up``.
-    ``scale`` (finished sums only): see :class:`RowScale`.
+    ``scale`` (finished sums only): see :class:`RowScale`.  ``activation`` (without ``pairs``, finished sums only):
+    ``"relu2"``: ``out`` holds the square of the sums' relu.
     """
     _check(a, "a", torch.bfloat16, 2)
     _check(w, "w", torch.bfloat16, 2)
     _check(out, "out")
+    _epilogue_code(pairs, activation)
     M, K = a.shape
     N = w.shape[0]
     if w.shape[1] != K:
@@ -324,7 +339,7 @@ def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, nsplit: int = 1
     ss, parts, inv_width, eps = _scale_args(scale, M)
     call(core(), "ap_gemm_tc", a.data_ptr(), w.data_ptr(), out.data_ptr(), dtype_code(out.dtype),
          M, N, K, K, K, N // 2 if pairs else N, nsplit, stride, 1 if reduce else 0,
-         (1 | ((_pairs_code(pairs) - 1) << 8)) if pairs else 0,
+         (1 | ((_pairs_code(pairs) - 1) << 8)) if pairs else EPILOGUE_ACTIVATIONS[activation] << 8,
          ss, parts, inv_width, eps, 0, 0, 0, 0, stream_handle())
 
 
@@ -408,14 +423,14 @@ def gemm_tc_dual(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
 
 
 def gemm_tc_pair(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, pairs: bool = False,
-                 share_tiles: bool = True) -> None:
+                 share_tiles: bool = True, activation: Optional[str] = None) -> None:
     """The tensor-core product on pairs of SMs (``tcgen05.mma.cta_group::2``), for many rows: two
     CTAs share a tile of 256 weight rows x up to 256 rows of ``a``, each loading half of either.
     With ``share_tiles`` a product of fewer tiles than half the pairs splits every tile's K among
     up to four pairs.
 
     ``pairs`` False: ``out[M,N] = a[M,K] @ w[N,K]^T``.  True: the rows of ``w [N,K]`` alternate
-    gate, up, gate, up ... and ``out[M,N/2] = silu(gate) * up``.
+    gate, up, gate, up ... and ``out[M,N/2] = silu(gate) * up``.  ``activation``: as for :func:`gemm_tc`.
     """
     _check(a, "a", torch.bfloat16, 2)
     _check(w, "w", torch.bfloat16, 2)
@@ -427,7 +442,7 @@ def gemm_tc_pair(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, pairs: boo
         raise KernelError(f"gemm_tc_pair: shapes disagree: a {tuple(a.shape)}, w {tuple(w.shape)}, out {tuple(out.shape)}")
     scratch = _scratch_for_persistent(a.device) if share_tiles else None
     call(core(), "ap_gemm_tc_pair", a.data_ptr(), w.data_ptr(), out.data_ptr(), dtype_code(out.dtype),
-         M, N, K, K, K, n_out, _pairs_code(pairs), scratch.data_ptr() if scratch is not None else 0,
+         M, N, K, K, K, n_out, _epilogue_code(pairs, activation), scratch.data_ptr() if scratch is not None else 0,
          scratch.numel() if scratch is not None else 0, stream_handle())
 
 
@@ -448,14 +463,14 @@ def _scratch_for_persistent(device: torch.device) -> torch.Tensor:
 
 
 def gemm_tc_persistent(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, pairs: bool = False,
-                       share_tiles: bool = True) -> None:
+                       share_tiles: bool = True, activation: Optional[str] = None) -> None:
     """The persistent tensor-core product for more than 64 rows: one CTA per SM walks the
     output tiles, and a tile is written out while the next one is being computed.  With
     ``share_tiles`` a product of fewer tiles than half the SMs splits every tile's K among
     several CTAs.
 
     ``pairs`` False: ``out[M,N] = a[M,K] @ w[N,K]^T``.  True: the rows of ``w [N,K]`` alternate
-    gate, up, gate, up ... and ``out[M,N/2] = silu(gate) * up``.
+    gate, up, gate, up ... and ``out[M,N/2] = silu(gate) * up``.  ``activation``: as for :func:`gemm_tc`.
     """
     _check(a, "a", torch.bfloat16, 2)
     _check(w, "w", torch.bfloat16, 2)
@@ -468,7 +483,7 @@ def gemm_tc_persistent(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, pair
                           f"out {tuple(out.shape)}")
     scratch = _scratch_for_persistent(a.device) if share_tiles else None
     call(core(), "ap_gemm_tc_persistent", a.data_ptr(), w.data_ptr(), out.data_ptr(), dtype_code(out.dtype),
-         M, N, K, K, K, n_out, _pairs_code(pairs), scratch.data_ptr() if scratch is not None else 0,
+         M, N, K, K, K, n_out, _epilogue_code(pairs, activation), scratch.data_ptr() if scratch is not None else 0,
          scratch.numel() if scratch is not None else 0, stream_handle())
 
 

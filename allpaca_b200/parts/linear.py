@@ -116,25 +116,36 @@ class Linear:
         return out
 
     @staticmethod
-    def tensor_core_product(a: torch.Tensor, w: torch.Tensor, target: torch.Tensor, scale=None) -> bool:
+    def tensor_core_product(a: torch.Tensor, w: torch.Tensor, target: torch.Tensor, scale=None,
+                            activation: Optional[str] = None) -> bool:
         """``target[T, N] = a[T, K] @ w[N, K]^T`` in bfloat16 on the tensor cores, by the kernel that
-        suits the shape; returns whether ``scale`` was applied (only the kernel for few rows can)."""
+        suits the shape; returns whether ``scale`` was applied (only the kernel for few rows can).
+        ``activation`` (``"relu2"``): of the sums, in the product's epilogue."""
         T, K = a.shape
         N = w.shape[0]
         nsplit = ops.gemm_tc_splits(T, N, K)
         if T > 64 and nsplit > 1:
             # up to 256 rows against few weight tiles: K slices in a cluster, as for decoding
-            ops.gemm_tc(a, w, target, nsplit, reduce=True)
+            ops.gemm_tc(a, w, target, nsplit, reduce=True, activation=activation)
         elif ops.gemm_tc_prefers_pair(T, N, K):
-            ops.gemm_tc_pair(a, w, target)
+            ops.gemm_tc_pair(a, w, target, activation=activation)
         elif T > 64 and ops.gemm_tc_prefers_persistent(T, N, K):
-            ops.gemm_tc_persistent(a, w, target)
-        elif nsplit == 1 and ops.gemm_tc_prefers_dual(T, N, K):
+            ops.gemm_tc_persistent(a, w, target, activation=activation)
+        elif nsplit == 1 and activation is None and ops.gemm_tc_prefers_dual(T, N, K):
             ops.gemm_tc_dual(a, w, target)
         else:
-            ops.gemm_tc(a, w, target, nsplit, reduce=nsplit > 1, scale=scale)
+            ops.gemm_tc(a, w, target, nsplit, reduce=nsplit > 1, scale=scale, activation=activation)
             return True
         return False
+
+    def forward_activated(self, a: torch.Tensor, buffer_name: str, activation: str) -> Optional[torch.Tensor]:
+        """``act(a W^T)`` in one kernel, ``[T, out]`` in the activation type; None where no product does that (the
+        caller then multiplies and activates separately)."""
+        if not self.uses_tensor_cores() or self.bias is not None or activation not in ops.EPILOGUE_ACTIVATIONS:
+            return None
+        out = self.env.workspace.get(buffer_name, (a.shape[0], self.out_features), self.env.dtype)
+        self.tensor_core_product(a, self.weight, out, activation=activation)
+        return out
 
     def forward_gated(self, a: torch.Tensor, buffer_name: str, scale=None, activation: str = "silu") -> Optional[torch.Tensor]:
         """For a weight whose rows alternate gate and up: ``act(a W_gate^T) * (a W_up^T)`` in one

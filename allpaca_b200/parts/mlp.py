@@ -98,7 +98,8 @@ class DenseActivation(FeedForward):
     (local tensor names of up and down, default ``("up", "down")``; a bias is ``<name>.b``).
 
     The first product leaves 32-bit sums; bias and activation act on those in one kernel and round once to
-    the activation type; the second product's bias is added to its 32-bit sums."""
+    the activation type (without biases the square of relu is applied in the product's epilogue on the tensor
+    cores); the second product's bias is added to its 32-bit sums."""
 
     def __init__(self, params, env: BuildEnv):
         super().__init__(params, env)
@@ -129,7 +130,9 @@ class DenseActivation(FeedForward):
 
     def forward(self, h: torch.Tensor, step) -> torch.Tensor:
         T = h.shape[0]
-        sums = self.up.forward(h, "ffn.up", "float32")
-        act = self.env.workspace.get("ffn.act", (T, self.inter), self.env.dtype)
-        ops.bias_act(sums, self.up_bias, act, self.activation)
+        act = self.up.forward_activated(h, "ffn.act", self.activation) if self.up_bias is None else None
+        if act is None:
+            sums = self.up.forward(h, "ffn.up", "float32")
+            act = self.env.workspace.get("ffn.act", (T, self.inter), self.env.dtype)
+            ops.bias_act(sums, self.up_bias, act, self.activation)
         return self.down.forward(act, "ffn.down", "delta")

@@ -174,15 +174,19 @@ class RoutedExperts(FeedForward):
             first = offsets.tolist()                                   # the step waits for the device here
             rows = ws.get("moe.rows", (pairs, self.hidden), torch.bfloat16)
             ops.moe_gather(h, rows, perm, self.top)
-            gu = ws.get("moe.gate_up", (pairs, self.first_rows), torch.bfloat16 if self.gated else torch.float32)
+            # without a gate the square of relu is applied in the products' epilogues; else by a pass over all pairs
+            fused = not self.gated and self.activation in ops.EPILOGUE_ACTIVATIONS
+            gu = y if fused else ws.get("moe.gate_up", (pairs, self.first_rows),
+                                        torch.bfloat16 if self.gated else torch.float32)
             for e in range(self.experts):
                 a, b = first[e], first[e + 1]
                 if b > a:
-                    Linear.tensor_core_product(rows[a:b], self.gate_up[e], gu[a:b])
+                    Linear.tensor_core_product(rows[a:b], self.gate_up[e], gu[a:b],
+                                               activation=self.activation if fused else None)
             if self.gated:
                 ops.gated_act(gu, y, self.activation, False, self.limit, self.alpha, self.shift,
                               row_scale=weight.view(-1) if on_input else None, scale_index=perm if on_input else None)
-            else:
+            elif not fused:
                 ops.bias_act(gu, None, y, self.activation)
             for e in range(self.experts):
                 a, b = first[e], first[e + 1]

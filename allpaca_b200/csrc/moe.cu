@@ -526,32 +526,26 @@ moe_rows_kernel(const bf16* __restrict__ A, long long lda, const bf16* __restric
     for (int r0 = 0; r0 < rows; r0 += ROWS_MAX) {
         const int R = min(ROWS_MAX, rows - r0);
         __syncthreads();
-        for (int i = threadIdx.x; i < ROWS_MAX * K8; i += 256) {
+        for (int i = threadIdx.x; i < R * K8; i += 256) {
             const int r = i / K8, c = i - r * K8;
-            uint4 v = make_uint4(0, 0, 0, 0);
-            if (r < R) {
-                const int src = FIRST ? perm[p0 + r0 + r] / top : p0 + r0 + r;
-                v = *reinterpret_cast<const uint4*>(A + (size_t)src * lda + c * 8);
-            }
-            *reinterpret_cast<uint4*>(a_s + (size_t)r * K + c * 8) = v;
+            const int src = FIRST ? perm[p0 + r0 + r] / top : p0 + r0 + r;
+            *reinterpret_cast<uint4*>(a_s + (size_t)r * K + c * 8) = *reinterpret_cast<const uint4*>(A + (size_t)src * lda + c * 8);
         }
         __syncthreads();
-        for (int cc = 0; cc < ROWS_COLS / 8; ++cc) {
+        // two weight rows at a time, so that what is read of the tile's rows serves both: a gate's and its up's, or (no
+        // gate) two neighbouring columns'
+        for (int cc = 0; cc < ROWS_COLS / 8; cc += GATED ? 1 : 2) {
             const int n = blockIdx.x * ROWS_COLS + warp * (ROWS_COLS / 8) + cc;
             if (n >= N) break;
-            float acc[ROWS_MAX], acc2[GATED ? ROWS_MAX : 1];
+            float acc[ROWS_MAX], acc2[ROWS_MAX];
 #pragma unroll
-            for (int r = 0; r < ROWS_MAX; ++r) {
-                acc[r] = 0.f;
-                if constexpr (GATED) acc2[r] = 0.f;
-            }
+            for (int r = 0; r < ROWS_MAX; ++r) acc[r] = acc2[r] = 0.f;
             const bf16* w1 = We + (size_t)n * K;
-            const bf16* w2 = We + (size_t)(N + n) * K;
+            const bf16* w2 = We + (size_t)(GATED ? N + n : min(n + 1, N - 1)) * K;
 #pragma unroll 4
             for (int k = lane * 8; k < K; k += 256) {
                 const uint4 wv = *reinterpret_cast<const uint4*>(w1 + k);
-                uint4 wv2 = make_uint4(0, 0, 0, 0);
-                if constexpr (GATED) wv2 = *reinterpret_cast<const uint4*>(w2 + k);
+                const uint4 wv2 = *reinterpret_cast<const uint4*>(w2 + k);
                 const __nv_bfloat162* wp = reinterpret_cast<const __nv_bfloat162*>(&wv);
                 const __nv_bfloat162* wp2 = reinterpret_cast<const __nv_bfloat162*>(&wv2);
                 float wf[8], wf2[8];
@@ -559,20 +553,19 @@ moe_rows_kernel(const bf16* __restrict__ A, long long lda, const bf16* __restric
                 for (int q = 0; q < 4; ++q) {
                     const float2 t = __bfloat1622float2(wp[q]);
                     wf[2 * q] = t.x; wf[2 * q + 1] = t.y;
-                    if constexpr (GATED) {
-                        const float2 u = __bfloat1622float2(wp2[q]);
-                        wf2[2 * q] = u.x; wf2[2 * q + 1] = u.y;
-                    }
+                    const float2 u = __bfloat1622float2(wp2[q]);
+                    wf2[2 * q] = u.x; wf2[2 * q + 1] = u.y;
                 }
 #pragma unroll
                 for (int r = 0; r < ROWS_MAX; ++r) {
+                    if (r >= R) break;
                     const uint4 av = *reinterpret_cast<const uint4*>(a_s + (size_t)r * K + k);
                     const __nv_bfloat162* ap = reinterpret_cast<const __nv_bfloat162*>(&av);
 #pragma unroll
                     for (int q = 0; q < 4; ++q) {
                         const float2 t = __bfloat1622float2(ap[q]);
                         acc[r] = fmaf(t.y, wf[2 * q + 1], fmaf(t.x, wf[2 * q], acc[r]));
-                        if constexpr (GATED) acc2[r] = fmaf(t.y, wf2[2 * q + 1], fmaf(t.x, wf2[2 * q], acc2[r]));
+                        acc2[r] = fmaf(t.y, wf2[2 * q + 1], fmaf(t.x, wf2[2 * q], acc2[r]));
                     }
                 }
             }
@@ -581,15 +574,19 @@ moe_rows_kernel(const bf16* __restrict__ A, long long lda, const bf16* __restric
             // sum is formed by the same tree as a butterfly over all lanes, and ends in the lanes whose bits 4, 3, 2
             // spell the row
             const int out_row = ((lane >> 4) & 1) * 4 + ((lane >> 3) & 1) * 2 + ((lane >> 2) & 1);
-            float v = moe_rows_sum8(acc, lane), v2 = 0.f;
-            if constexpr (GATED) v2 = moe_rows_sum8(acc2, lane);
+            float v = moe_rows_sum8(acc, lane), v2 = moe_rows_sum8(acc2, lane);
             if ((lane & 3) == 0 && out_row < R) {
                 if constexpr (FIRST) {
                     const float sc = pair_scale ? pair_scale[perm[p0 + r0 + out_row]] : 1.0f;
                     if constexpr (GATED) v = gated_activation(v * sc, v2 * sc, act, limit, alpha, shift);
-                    else v = gated_activation(v * sc, 1.0f, act, 0.f, 0.f, 0.f);
+                    else {
+                        v = gated_activation(v * sc, 1.0f, act, 0.f, 0.f, 0.f);
+                        v2 = gated_activation(v2 * sc, 1.0f, act, 0.f, 0.f, 0.f);
+                    }
                 }
-                C[(size_t)(p0 + r0 + out_row) * ldc + n] = ap_from_float<TO>(v);
+                TO* c = C + (size_t)(p0 + r0 + out_row) * ldc + n;
+                c[0] = ap_from_float<TO>(v);
+                if (!GATED && n + 1 < N) c[1] = ap_from_float<TO>(v2);
             }
         }
     }

@@ -406,3 +406,51 @@ def test_experts_without_a_gate_and_a_shared_one(dtype, tol, W, F, E, top, count
     if shared:
         mlp["shared"] = {"ff": shared}
     close(got, plain.experts({"x." + k: v.double() for k, v in w.items()}, "x.", mlp, h.double()), tol, "routed feed-forward")
+
+
+@pytest.mark.parametrize("M,N,K", [(1, 40, 64), (8, 1024, 2048), (37, 200, 96), (64, 128, 4096), (100, 96, 320), (200, 256, 512),
+                                   (300, 1024, 256), (700, 136, 128), (2048, 1024, 512), (520, 4096, 6400)])
+@pytest.mark.parametrize("out_dtype", [torch.bfloat16, torch.float32])
+def test_squared_relu_in_the_products_epilogue(M, N, K, out_dtype):
+    """Whatever kernel the shape is given to: slices of K in a cluster, one tile to a CTA, persistent, pairs of SMs."""
+    from allpaca_b200 import ops
+    from allpaca_b200.parts.linear import Linear
+    g = torch.Generator().manual_seed(M + N)
+    a, w = torch.randn(M, K, generator=g).to(torch.bfloat16), (torch.randn(N, K, generator=g) * K ** -0.5).to(torch.bfloat16)
+    z = torch.relu(a.double() @ w.double().T)
+    ad, wd = a.to(DEV), w.to(DEV)
+    out = torch.full((M, N), float("nan"), dtype=out_dtype, device=DEV)
+    Linear.tensor_core_product(ad, wd, out, activation="relu2")
+    tol = 3e-5 if out_dtype == torch.float32 else 1e-2
+    close(out, z * z, tol, "the kernel of the shape")
+    if M > 64:
+        for product in (ops.gemm_tc_persistent, ops.gemm_tc_pair):
+            out.fill_(float("nan"))
+            product(ad, wd, out, activation="relu2")
+            close(out, z * z, tol, product.__name__)
+    ops.check_kernel_status()
+
+
+@pytest.mark.parametrize("W", [64, 42, 320, 2048, 4100, 8192, 20000])
+@pytest.mark.parametrize("T", [3, 700])
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_one_stream_between_two_norms(W, T, dtype):
+    """A sublayer's normed result into the stream and the norm of what the next one reads, in steps of few rows and many;
+    chosen rows leave the stream alone."""
+    from allpaca_b200 import ops
+    g = torch.Generator().manual_seed(W + T)
+    x, d = torch.randn(T, 1, W, generator=g), 5 * torch.randn(1, T, W, generator=g)
+    w, sw = 1 + 0.2 * torch.randn(W, generator=g), torch.randn(1, W, generator=g)
+    one = torch.ones(1, device=DEV)
+    want = x.double()[:, 0] + plain.rms(d.double()[0], 0.3) * sw.double()
+    read = plain.rms(want, 1e-5) * w.double()
+    kw = dict(delta=d.to(DEV), out_w=one, mix=one.view(1, 1), slice_weight=sw.to(DEV), slice_eps=0.3)
+    tol = 2e-5 if dtype == torch.float32 else 1e-2
+    xd, out = x.to(DEV), torch.empty(T, W, dtype=dtype, device=DEV)
+    ops.stream_norm(xd, one, w.to(DEV), 1e-5, out, **kw)
+    close(xd[:, 0], want, 2e-5, "the stream")
+    close(out, read, tol, "what the sublayer reads")
+    xd, out = x.to(DEV), torch.empty(2, W, dtype=dtype, device=DEV)
+    ops.stream_norm(xd, one, w.to(DEV), 1e-5, out, rows=i32([T - 1, 0]), **kw)
+    close(out, read[[T - 1, 0]], tol, "chosen rows")
+    assert torch.equal(xd.cpu(), x)

@@ -7,6 +7,7 @@
     python -m allpaca_b200.bench_kernels latent-prefill --tokens 2048             # a prompt on per-head keys and values
     python -m allpaca_b200.bench_kernels stream --rows 2048 --width 2048          # norms without statistics, token shift, depth average
     python -m allpaca_b200.bench_kernels recurrent --rows 2048 --seqs 1          # linear-attention recurrences, the norm after a gated sum
+    python -m allpaca_b200.bench_kernels experts --rows 8                        # routed experts' products at few rows
     python -m allpaca_b200.bench_kernels versus-reference      # a table: ours against the reference's own kernels
 
 Each call works on the next of several copies of its large operand (together larger than
@@ -552,6 +553,41 @@ def bench_recurrent(args) -> dict:
     return res
 
 
+def bench_experts(args) -> dict:
+    """The grouped products of routed experts for ``--rows`` rows that each use ``--top`` of ``--experts`` (drawn at
+    random): the first product with a gate (SiLU) and without (the square of relu), the second one, and the sum of a row's
+    results with and without something to add to, each beside the bytes of the experts that are used."""
+    from allpaca_b200 import ops
+    T, E, top, F, H = args.rows, args.experts, args.top, args.ff, args.width
+    dev, pairs = "cuda", args.rows * args.top
+    g = torch.Generator().manual_seed(1)
+    chosen = torch.stack([torch.randperm(E, generator=g)[:top] for _ in range(T)]).to(torch.int32).to(dev)
+    used = int(chosen.unique().numel())
+    perm, place = (torch.empty(pairs, dtype=torch.int32, device=dev) for _ in range(2))
+    tiles = torch.empty(ops.moe_max_tiles(pairs, E) + 1, 3, dtype=torch.int32, device=dev)
+    ops.moe_sort(chosen, perm, place, tiles, E)
+    copies = max(2, int(math.ceil(300e6 / (E * F * H * 2))))
+    gate_up = [torch.randn(E, 2 * F, H, device=dev).to(torch.bfloat16) * 0.02 for _ in range(copies)]
+    up = [w[:, :F].contiguous() for w in gate_up]
+    down = [torch.randn(E, H, F, device=dev).to(torch.bfloat16) * 0.02 for _ in range(copies)]
+    a = torch.randn(T, H, device=dev).to(torch.bfloat16)
+    y, o = torch.empty(pairs, F, device=dev, dtype=torch.bfloat16), torch.empty(pairs, H, device=dev)
+    weight, delta, base = torch.rand(T, top, device=dev), torch.empty(T, H, device=dev), torch.randn(T, H, device=dev)
+    one = used * F * H * 2
+    cases = {
+        "first product, gated": (lambda i: ops.moe_gate_up(a, gate_up[i % copies], y, perm, top, tiles, "silu"), 2 * one),
+        "first product, no gate": (lambda i: ops.moe_gate_up(a, up[i % copies], y, perm, top, tiles, "relu2", gated=False), one),
+        "second product": (lambda i: ops.moe_down(y, down[i % copies], o, tiles), one),
+        "moe_combine": (lambda i: ops.moe_combine(o, place, weight, delta), pairs * H * 4 + T * H * 4),
+        "moe_combine on a base": (lambda i: ops.moe_combine(o, place, weight, delta, base=base), pairs * H * 4 + T * H * 8),
+    }
+    res = {"rows": T, "experts": E, "top": top, "ff": F, "width": H, "experts_used": used}
+    for name, (fn, nbytes) in cases.items():
+        us = _time(fn, args.iters, args.warmup, not args.no_graph)
+        res[name] = {"us": round(us, 2), "MB": round(nbytes / 1e6, 1), "GBps": round(nbytes / us / 1e3, 1)}
+    return res
+
+
 def bench_sampling(args) -> dict:
     """The choice of the next token for ``--rows`` rows of logits over ``--vocab`` entries."""
     from allpaca_b200 import ops
@@ -669,13 +705,22 @@ def main(argv=None) -> int:
     s.add_argument("--groups", type=int, default=4)
     s.add_argument("--streams", type=int, default=4)
     s.add_argument("--token-by-token", action="store_true", help="never eight tokens at a time")
+    s = sub.add_parser("experts")
+    s.add_argument("--iters", type=int, default=50)
+    s.add_argument("--warmup", type=int, default=5)
+    s.add_argument("--no-graph", action="store_true", help="launch from the host (for ncu)")
+    s.add_argument("--rows", type=int, default=8)
+    s.add_argument("--experts", type=int, default=16)
+    s.add_argument("--top", type=int, default=4)
+    s.add_argument("--ff", type=int, default=1024)
+    s.add_argument("--width", type=int, default=2048)
     s = sub.add_parser("versus-reference")
     s.add_argument("--iters", type=int, default=20)
     s.add_argument("--warmup", type=int, default=3)
     args = p.parse_args(argv)
     fn = {"gemm": bench_gemm, "attention": bench_attention, "prefill-attention": bench_prefill_attention,
           "sampling": bench_sampling, "versus-reference": bench_versus_reference,
-          "stream": bench_stream, "recurrent": bench_recurrent, "latent-decode": bench_latent_decode, "latent-prefill": bench_latent_prefill}[args.what]
+          "stream": bench_stream, "recurrent": bench_recurrent, "experts": bench_experts, "latent-decode": bench_latent_decode, "latent-prefill": bench_latent_prefill}[args.what]
     print(json.dumps(fn(args)))
     return 0
 

@@ -264,7 +264,7 @@ def test_readers_of_one_layers_keys_behind_windows_of_their_own(dtype, tol, H, G
             close(out.float().reshape(-1, H, E), torch.cat(want), tol, ("window", w, single))
 
 
-@pytest.mark.parametrize("H,R,E,P,window", [(8, 64, 16, 16, 40), (5, 32, 8, 8, 19), (4, 128, 24, 16, 33), (16, 512, 64, 32, 500),
+@pytest.mark.parametrize("H,R,E,P,window", [(7, 72, 24, 16, 45), (5, 32, 8, 8, 19), (4, 128, 24, 16, 33), (16, 512, 64, 32, 500),
                                             (3, 18, 6, 8, 11), (2, 62, 2, 64, 1)])
 @pytest.mark.parametrize("dtype,tol", [(torch.float32, 3e-5), (torch.bfloat16, 2e-2)])
 def test_records_of_a_latent_and_a_rotated_part_behind_a_window(dtype, tol, H, R, E, P, window):
@@ -313,7 +313,7 @@ def test_records_of_a_latent_and_a_rotated_part_behind_a_window(dtype, tol, H, R
 
 
 # ---- routed experts -----------------------------------------------------------------------------
-@pytest.mark.parametrize("E,top,count,keep", [(12, 4, 2, 1), (10, 3, 5, 2), (256, 16, 8, 3), (9, 2, 9, 2), (64, 1, 1, 1),
+@pytest.mark.parametrize("E,top,count,keep", [(14, 3, 2, 1), (10, 3, 5, 2), (256, 16, 8, 3), (9, 2, 9, 2), (64, 1, 1, 1),
                                               (33, 5, 3, 3), (6, 2, 3, 1), (200, 7, 40, 4), (128, 8, 128, 8), (1, 1, 1, 1)])
 @pytest.mark.parametrize("T", [3, 600])
 def test_choice_among_the_best_groups(E, top, count, keep, T):
